@@ -71,7 +71,7 @@ B200_DEVICE void mbar_wait(uint32_t bar, uint32_t parity)
     while (!mbar_try_wait(bar, parity)) {}
 }
 
-// 1-D bulk async copy global -> shared, completion signalled on an mbarrier (SASS: UBLKCP).
+// 1-D bulk async copy global -> shared, completion signalled on an mbarrier.
 B200_DEVICE void bulk_g2s(uint32_t dst_smem, const void* src, uint32_t bytes, uint32_t bar)
 {
     asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(

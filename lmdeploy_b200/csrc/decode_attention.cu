@@ -201,7 +201,7 @@ __global__ void __launch_bounds__(128) kv_prologue_kernel(const PrologueParams p
             if (di + 2 * i < p.rope.dim) {
                 const T c = Ops::from_f32(cs[i].x), s = Ops::from_f32(cs[i].y);
                 const T a = x[2 * i], bb = x[2 * i + 1];
-                // the reference binary contracts `c*x0 - s*x1` to HMUL2 + HFMA2 (SASS of oracle/_ref)
+                // `c*x0 - s*x1` as one product and one fused multiply-add: what nvcc's default -fmad makes of the reference's source
                 x[2 * i]     = Ops::fma(c, a, Ops::neg(Ops::mul(s, bb)));
                 x[2 * i + 1] = Ops::fma(c, bb, Ops::mul(s, a));
             }

@@ -137,8 +137,8 @@ __device__ __forceinline__ float2 rope_cos_sin(const RopeConst& r, int idx, int 
 }
 
 
-// bias + RoPE of 4 consecutive dims [di, di + 4) of one head vector, T arithmetic exactly as the reference binary's
-// (rotary_embedding.h:168-181 compiled with --use_fast_math: `c*x0 - s*x1` contracted to HMUL2 + HFMA2)
+// bias + RoPE of 4 consecutive dims [di, di + 4) of one head vector, T arithmetic as the reference's release build
+// (rotary_embedding.h:168-181 compiled with --use_fast_math: `c*x0 - s*x1` as a product and a fused multiply-add)
 template<class T>
 __device__ __forceinline__ void rope_rotate4(T (&x)[4], const float2 (&cs)[2], const RopeConst& rope, int di)
 {

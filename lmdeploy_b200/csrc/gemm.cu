@@ -292,7 +292,7 @@ static Plan make_plan(int fmt, int MT, int N, int K, bool need_split = false)
         pl.nx = std::max(2, std::min(kMaxX, (budget - pl.nw * wslot) / XB));
     }
     // u4: a W ring of exactly 8 slots selects the de-quantisation loop that is unrolled over one lap of the ring (all ring
-    // positions compile-time constants, 126 instead of 162 instructions per k-group); trade X slots for it while >= 3 remain
+    // positions compile-time constants); trade X slots for it while >= 3 remain
     if (fmt == kU4 && pl.nw < 8) {
         for (int nx = pl.nx - 1; nx >= 3; --nx) {
             if ((budget - nx * XB) / wslot >= 8) {

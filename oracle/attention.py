@@ -148,9 +148,9 @@ def rope_inv_freq(rope: RopeParam):
 
 def apply_rope(x, pos, rope: RopeParam, dtype):
     """x: [..., D] float32 (exact in T); pos: int array broadcastable to x[..., 0].
-    Adjacent-pair rotation computed in T (rotary_embedding.h:168-181).  The reference binary contracts each
-    `(T)c*x0 - (T)s*x1` into HMUL2 + HFMA2 (mul.f16 / sub.f16 carry no .rn, so ptxas may fuse; checked in the SASS of
-    oracle/_ref: decoding_sm80_128 / ProcessKV_v2):  x0' = fma(c, x0, -RN(s*x1)) ; x1' = fma(c, x1, RN(s*x0))."""
+    Adjacent-pair rotation computed in T (rotary_embedding.h:168-181).  Each `(T)c*x0 - (T)s*x1` of
+    the reference's source is one product and one fused multiply-add (nvcc's default -fmad; the recorded outputs of the
+    reference's kernels agree bit for bit):  x0' = fma(c, x0, -RN(s*x1)) ; x1' = fma(c, x1, RN(s*x0))."""
     if rope.type == ROPE_NULL:
         return f32(x).copy()
     kp = rope.kernel_params()

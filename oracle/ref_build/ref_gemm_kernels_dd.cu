@@ -5,8 +5,7 @@
 // (arch/config_sm80_s16816.h:108-121).  Most of them stream the weights with PolicyB = cache_policy::Stream, i.e.
 // cp.async ... .L2::cache_hint with a createpolicy.fractional.L2::evict_first descriptor (iterator_sm80.h:145-149,
 // cp_async.h:127-137).  With this image's toolchain (ptxas 12.9.86, and the 580 driver's JIT on compute_80 PTX alike)
-// that instruction is encoded as `LDGSTS... desc[UR1]` and a B200 raises "illegal instruction" on it
-// (compute-sanitizer, profiles/r02_ref_gemm_illegal_instruction.md) -- the reference's own default dispatch picks such
+// a B200 raises "illegal instruction" on it (compute-sanitizer, profiles/r02_ref_gemm_illegal_instruction.md) -- the reference's own default dispatch picks such
 // a kernel at m = 1 and m = 64, so its GEMM cannot run here as built.
 //
 // This translation unit registers the SAME templates at the SAME tile shapes with the evict-first hint switched off

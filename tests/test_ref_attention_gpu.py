@@ -4,7 +4,7 @@ same device buffers as ours.  This is what pins the numpy oracle and our kernels
 reference stores no golden vectors for this path).
 
 Bars (rope.exact_math = 0, i.e. the arithmetic of the reference's release build: ex2.approx / sin.approx / cos.approx
-and the mul+fma contraction its SASS shows):
+and the mul+fma contraction of nvcc's default -fmad):
   * every byte the prologue / ProcessKV writes to the KV pages (K, V, scale, zero): BIT-IDENTICAL;
   * attention output: |ours - reference| <= 2e-3 (fp16) / 1.6e-2 (bf16) on identical cache contents (split counts
     and the fp32 summation order differ by design).

@@ -1,5 +1,5 @@
 // Development tool (not on the product path): two questions the GEMM / attention producers hinge on.
-//  (1) What does ISSUING a 1-D bulk copy (cp.async.bulk, SASS UBLKCP) cost the issuing thread, and does spreading the
+//  (1) What does ISSUING a 1-D bulk copy (cp.async.bulk) cost the issuing thread, and does spreading the
 //      issues over the lanes of a warp hide it?  (tools/gemm_trace timelines show ~300 cycles between back-to-back
 //      issues from one lane; the attention producer got faster when ten lanes issued one copy each.)
 //  (2) What per-SM and aggregate ingest rate do bulk copies reach as a function of copy size, copies in flight, and
