@@ -3,7 +3,9 @@
  * grouped key/value heads, residual add + RMS norm, learned positions; parallel blocks with two norms, convolved rotary
  * attention whose values are its keys, a selective state-space mixer, sigmoid-routed experts; parallel blocks with one norm
  * and a token shift, two mixers side by side, chunked rotary attention with scores mixed across heads, a recurrence with a
- * decay per key channel and token, a router that chooses among groups of experts) for sm_100a.
+ * decay per key channel and token, a router that chooses among groups of experts; blocks that norm a sublayer's input and its
+ * output, queries that grow with their position, gated linear attention, a real-gated diagonal recurrence, a router whose
+ * softmax runs over the chosen experts) for sm_100a.
  *
  * Conventions shared by all entries: raw device pointers, sizes as int, `stream` a cudaStream_t, return 0 on success, a
  * negative b200h_status for refused arguments, a positive cudaError_t for a failed launch; b200h_last_error() says why.
@@ -20,56 +22,6 @@
 #define B200H_API extern "C" __attribute__((visibility("default")))
 #else
 #define B200H_API
-
-/* ---- parallel blocks with one norm and a token shift, side-by-side mixers, recurrence with a decay per channel and token ---- */
-
-/* out[t] = table[tokens[t]] + second[row] (float), row = (previous token * mul_prev + tokens[t] * mul_cur) mod buckets, or `buckets`
- * (the table's last row) at position 0.  The token before an entry's first row is the int at prev + seq_slot[s] * slot_stride (in
- * a float's place), which then becomes the entry's last token of this step. */
-B200H_API int b200h_embed_hashed(const void* tokens, const void* table, const void* second, int buckets, int mul_prev, int mul_cur, void* prev,
-                                 int64_t slot_stride, const void* tok_seq, const void* tok_pos, const void* cu_q, const void* seq_slot,
-                                 void* out, int n, int batch, int width, int dtype, void* stream);
-
-/* x[t] += branch_scale * (left[t] / rms(left[t]) * wl + right[t] / rms(right[t]) * wr) + sum_p ff[t, p]; then, if w is given,
- * hf[t] = x[t] / rms(x[t]) * w (float) and h[t] the same as T.  left, right: T [n, width] (both or neither) with wl, wr float
- * [width]; ff: T (or float when ff_is_f32) [n, parts, width] or NULL; h, hf optional. */
-B200H_API int b200h_branch_residual_norm(void* x, const void* left, const void* right, const void* wl, const void* wr, float branch_scale,
-                                         const void* ff, int ff_is_f32, int parts, const void* w, int n, int width, float eps, void* h,
-                                         void* hf, int dtype, void* stream);
-
-/* Token shift of normed rows h (float [n, width]): a[t] = h[t] + (h[t-1] - h[t]) * shift (shift float [width] or NULL: a = h), and
- * for m < nmu blends[m][t] = a[t] + (a[t-1] - a[t]) * mu[m] (mu float [nmu, width]; a, blends T, blends [nmu, n, width]; a optional).
- * The rows before an entry's first come from its state (float [2, width] = its last h and a at state + seq_slot[s] * slot_stride;
- * zeros at a sequence's start), which is then advanced by the step. */
-B200H_API int b200h_token_shift(const void* h, const void* shift, const void* mu, int nmu, void* state, int64_t slot_stride,
-                                const void* tok_seq, const void* cu_q, const void* seq_slot, int n, int batch, int width, void* a,
-                                void* blends, int dtype, void* stream);
-
-/* Per head, S a [dim, vdim] float matrix per sequence:  w_t = exp(-exp(d_t + w0)) per key channel;
- * out_t = (S + diag(bonus) k_t v_t^T)^T r_t;  S <- diag(w_t) S + k_t v_t^T.  r, k (heads * dim columns) and v (heads * vdim) are T
- * with row stride ld; d float [n, heads * dim]; w0, bonus float [heads * dim]; state float [heads, vdim, dim] at state + seq_slot[s] *
- * slot_stride, read and advanced; decay: float [n, heads * dim] scratch; out float [n, heads * vdim]. */
-B200H_API int b200h_channel_decay_scan(const void* r, const void* k, const void* v, int64_t ld, const void* d, const void* w0,
-                                       const void* bonus, void* state, int64_t slot_stride, const void* cu_q, const void* seq_slot, int n,
-                                       int batch, int heads, int dim, int vdim, void* decay, void* out, int dtype, void* stream);
-
-/* y[t] = unit_rms_per_group(o[t]) * w * act(gate[t]) as T: the norm BEFORE the gate; o float [n, count], `groups` equal parts,
- * gate T with row stride ld_gate; act 0 sigmoid, 1 silu. */
-B200H_API int b200h_group_norm_gate(const void* o, const void* w, const void* gate, int64_t ld_gate, int n, int count, int groups, int act,
-                                    float eps, void* y, int dtype, void* stream);
-
-/* x <- z > 0 ? softplus(p) z^2 + z / 2 : (1/2 + softplus(q)) (exp(z) - 1 - z) + z / 2 in place (T); params = {p, q} floats on the device. */
-B200H_API int b200h_xielu(void* x, int64_t count, const void* params, int dtype, void* stream);
-
-/* x <- tanh(x) in place (T). */
-B200H_API int b200h_tanh(void* x, int64_t count, int dtype, void* stream);
-
-/* Router with sigmoid scores s and groups of neighbouring experts: choice score = s + correction (float [experts] or NULL); a
- * group's score = the sum of its group_top largest choice scores; only experts of the `keep` best of `groups` equal groups can be
- * chosen; ids = the `top` largest choice scores; wts = the chosen s (without correction), / (their sum + 1e-20) if renorm, * scale. */
-B200H_API int b200h_route_grouped(const void* x, int x_dtype, const void* router, const void* correction, int n, int width, int experts,
-                                  int top, int groups, int keep, int group_top, int renorm, float scale, void* ids, void* wts, void* stream);
-
 #endif
 
 #define B200H_BF16 1
@@ -160,10 +112,11 @@ B200H_API int b200h_gated_rms(const void* o, const void* w, const void* gate, in
 
 /* softmax(router x) over all experts; ids / wts [n, top]: the top largest and their scores. */
 B200H_API int b200h_route(const void* x, const void* router, int n, int width, int experts, int top, void* ids, void* wts, void* stream);
-/* The same with x as float or T (x_dtype) and a choice of scores: score_fn 0 = softmax over all experts, 1 = sigmoid of every
- * logit on its own (the weights are the chosen experts' sigmoids, not renormalised). */
-B200H_API int b200h_route_scored(const void* x, int x_dtype, const void* router, int n, int width, int experts, int top, int score_fn,
-                                 void* ids, void* wts, void* stream);
+/* The same with x as float or T (x_dtype), logits = router x + bias (float [experts] or NULL) and a choice of scores: score_fn 0 =
+ * softmax over all experts, 1 = sigmoid of every logit on its own (the weights are the chosen experts' sigmoids, not renormalised),
+ * 2 = softmax over the `top` chosen logits only. */
+B200H_API int b200h_route_scored(const void* x, int x_dtype, const void* router, const void* bias, int n, int width, int experts, int top,
+                                 int score_fn, void* ids, void* wts, void* stream);
 
 /* Routed experts for a step of few rows (an expert's weights are read once for all rows that chose it), e = ids[t, k], w = wts[t, k]:
  *   act 0, scale_input 0:  out[t, k] = w * down_e (silu(gate_e x[t]) * (up_e x[t]))
@@ -253,6 +206,8 @@ typedef struct b200h_window_args {
     int chunk;               /* > 0: a query sees only keys j with j / chunk == i / chunk (chunks counted from position 0) */
     int talk_scores;         /* 1: talk mixes the heads' SCORES before the softmax (s_h <- sum_g talk[h, g] * s_g) instead of their weights */
     int gate_heads;          /* 1: gate is T [n, ld_gate] with ONE column per head instead of one per output column */
+    float q_temp_coef;       /* the prep entries multiply a query at position p by 1 + q_temp_coef * ln(1 + floor((p + 1) / q_temp_every)), */
+    double q_temp_every;     /* after bias, norm and rotation; q_temp_every 0: by one */
 } b200h_window_args;
 /* Bias, norm of query and key, cache store of key and value (fills qn). */
 B200H_API int b200h_window_prep(const b200h_window_args* args);
@@ -373,5 +328,66 @@ B200H_API int b200h_tanh(void* x, int64_t count, int dtype, void* stream);
  * chosen; ids = the `top` largest choice scores; wts = the chosen s (without correction), / (their sum + 1e-20) if renorm, * scale. */
 B200H_API int b200h_route_grouped(const void* x, int x_dtype, const void* router, const void* correction, int n, int width, int experts,
                                   int top, int groups, int keep, int group_top, int renorm, float scale, void* ids, void* wts, void* stream);
+
+/* ---- blocks with a norm before and after each sublayer, gated linear attention, real-gated diagonal recurrence ---- */
+
+/* y[t] = branch_scale * (left[t] / rms(left[t]) * wl + right[t] / rms(right[t]) * wr) + m[t] + sum_p ff[t, p];
+ * x[t] += y[t] / rms(y[t]) * w_post;  then, if w_next is given, hf[t] = x[t] / rms(x[t]) * w_next (float) and h[t] the same as T.
+ * left, right: T [n, width] (both or neither) with wl, wr float [width]; m: T [n, width] or NULL; ff: float [n, parts, width] or NULL;
+ * with none of them the stream is only normed.  h, hf optional. */
+B200H_API int b200h_normed_residual_norm(void* x, const void* left, const void* right, const void* wl, const void* wr, float branch_scale,
+                                         const void* m, const void* ff, int parts, const void* w_post, const void* w_next, int n, int width,
+                                         float eps, void* h, void* hf, int dtype, void* stream);
+
+/* decay[t, c] = sigmoid(sum_k a[k, c] * low[t, k] + bias[c]) ^ (1 / tau) as float [n, channels]; low T [n, rank] with row stride ld, a T
+ * [rank, channels], bias float [channels]. */
+B200H_API int b200h_low_rank_decay(const void* low, int64_t ld, const void* a, const void* bias, int n, int channels, int rank, float tau,
+                                   void* decay, int dtype, void* stream);
+
+/* Per head, S a [dim, vdim] float matrix per sequence:  S <- diag(decay_t) S + k_t v_t^T;  out_t = S^T (q_scale * q_t), read after the
+ * update.  q, k (heads * dim columns) and v (heads * vdim) are T with row stride ld; decay float [n, heads * dim]; state float [heads,
+ * vdim, dim] at state + seq_slot[s] * slot_stride, read and advanced; out float [n, heads * vdim]. */
+B200H_API int b200h_gated_linear_scan(const void* q, const void* k, const void* v, int64_t ld, float q_scale, const void* decay, void* state,
+                                      int64_t slot_stride, const void* cu_q, const void* seq_slot, int batch, int heads, int dim, int vdim,
+                                      void* out, int dtype, void* stream);
+
+/* One real-gated diagonal recurrence of `width` channels for one step.  x, y: T columns of a projection with row stride ld, before their
+ * biases.  b200h_gated_conv:  u[t, c] = conv_bias[c] + sum_j conv[c, j] * (x + x_bias)[t - taps + 1 + j, c] as T [n, width]; inputs
+ * before an entry's first row come from conv_state, zeros at a sequence's start.  b200h_real_gated_scan, with the gates'
+ * pre-activations z float [blocks, n, 2 * (width / blocks)] (part b of the channels: the decay gates' columns, then the input gates'):
+ *   r = sigmoid(z_r + r_bias), i = sigmoid(z_i + i_bias), log a = -rate * r * softplus(lam), S <- a S + sqrt(1 - a^2) * i * u,
+ *   out[t] = S * gelu_tanh(y + y_bias) as T [n, width];
+ * it advances S (float [width] at state + seq_slot[s] * slot_stride) and then conv_state (float [taps - 1, width], same stride: the last
+ * taps - 1 biased inputs, oldest first). */
+typedef struct b200h_rglru_args {
+    int n, batch, width, blocks, taps;
+    float rate;
+    const void* x;
+    const void* y;
+    int64_t ld;
+    const void* x_bias;      /* float [width] or NULL */
+    const void* y_bias;      /* float [width] or NULL */
+    const void* conv;        /* float [width, taps] */
+    const void* conv_bias;   /* float [width] or NULL */
+    void* u;                 /* T [n, width]: out of b200h_gated_conv */
+    const void* z;
+    const void* r_bias;      /* float [width] or NULL */
+    const void* i_bias;      /* float [width] or NULL */
+    const void* lam;         /* float [width] */
+    void* conv_state;
+    void* state;
+    int64_t slot_stride;
+    void* out;
+    const void* tok_seq;     /* int [n] */
+    const void* cu_q;        /* int [batch + 1] */
+    const void* seq_slot;    /* int [batch] */
+    int dtype;
+    void* stream;
+} b200h_rglru_args;
+B200H_API int b200h_gated_conv(const b200h_rglru_args* args);
+B200H_API int b200h_real_gated_scan(const b200h_rglru_args* args);
+
+/* out[t, i] = silu(gu[t, i]) * gu[t, cols + i] as T [n, cols]; gu T [n, 2 * cols]: between the stacked gate | up product and the down product. */
+B200H_API int b200h_silu_mul_rows(const void* gu, int n, int cols, void* out, int dtype, void* stream);
 
 #endif

@@ -49,7 +49,7 @@ class WindowArgs(C.Structure):
         ("ml", C.c_void_p), ("o_part", C.c_void_p), ("scores", C.c_void_p), ("score_ld", C.c_int64), ("y", C.c_void_p),
         ("tok_seq", C.c_void_p), ("tok_pos", C.c_void_p), ("block_ptrs", C.c_void_p), ("cu_blocks", C.c_void_p),
         ("layer_off", C.c_int64), ("v_off", C.c_int64), ("dtype", C.c_int), ("stream", C.c_void_p), ("sink", C.c_void_p),
-        ("chunk", C.c_int), ("talk_scores", C.c_int), ("gate_heads", C.c_int),
+        ("chunk", C.c_int), ("talk_scores", C.c_int), ("gate_heads", C.c_int), ("q_temp_coef", C.c_float), ("q_temp_every", C.c_double),
     ]
 
 
@@ -65,7 +65,18 @@ class ConvPrepArgs(C.Structure):
     ]
 
 
-SCORE_FN = {"softmax": 0, "sigmoid": 1}
+class RgLruArgs(C.Structure):
+    """b200h_rglru_args."""
+    _fields_ = [
+        ("n", C.c_int), ("batch", C.c_int), ("width", C.c_int), ("blocks", C.c_int), ("taps", C.c_int), ("rate", C.c_float),
+        ("x", C.c_void_p), ("y", C.c_void_p), ("ld", C.c_int64), ("x_bias", C.c_void_p), ("y_bias", C.c_void_p), ("conv", C.c_void_p),
+        ("conv_bias", C.c_void_p), ("u", C.c_void_p), ("z", C.c_void_p), ("r_bias", C.c_void_p), ("i_bias", C.c_void_p), ("lam", C.c_void_p),
+        ("conv_state", C.c_void_p), ("state", C.c_void_p), ("slot_stride", C.c_int64), ("out", C.c_void_p),
+        ("tok_seq", C.c_void_p), ("cu_q", C.c_void_p), ("seq_slot", C.c_void_p), ("dtype", C.c_int), ("stream", C.c_void_p),
+    ]
+
+
+SCORE_FN = {"softmax": 0, "sigmoid": 1, "softmax_chosen": 2}
 GATE_ACT = {"sigmoid": 0, "silu": 1}
 EXPERT_ACT = {"silu_gate": 0, "relu2": 1}
 
@@ -105,7 +116,7 @@ def load():
     lib.b200h_relu2.argtypes = [P, L64, I, P]
     lib.b200h_window_prep.argtypes = [C.POINTER(WindowArgs)]
     lib.b200h_window_attention.argtypes = [C.POINTER(WindowArgs)]
-    lib.b200h_route_scored.argtypes = [P, I, P, I, I, I, I, I, P, P, P]
+    lib.b200h_route_scored.argtypes = [P, I, P, P, I, I, I, I, I, P, P, P]
     lib.b200h_parallel_residual_norm.argtypes = [P, P, P, I, F, P, P, P, P, I, I, F, P, P, P, I, P]
     lib.b200h_short_conv.argtypes = [P, L64, P, P, I, P, L64, P, P, P, P, I, I, I, I, I, P]
     lib.b200h_ssm_scan.argtypes = [P, P, L64, P, P, P, P, L64, P, P, I, I, I, I, I, I, P, P, I, P]
@@ -122,6 +133,12 @@ def load():
     lib.b200h_xielu.argtypes = [P, L64, P, I, P]
     lib.b200h_tanh.argtypes = [P, L64, I, P]
     lib.b200h_route_grouped.argtypes = [P, I, P, P, I, I, I, I, I, I, I, I, F, P, P, P]
+    lib.b200h_normed_residual_norm.argtypes = [P, P, P, P, P, F, P, P, I, P, P, I, I, F, P, P, I, P]
+    lib.b200h_low_rank_decay.argtypes = [P, L64, P, P, I, I, I, F, P, I, P]
+    lib.b200h_gated_linear_scan.argtypes = [P, P, P, L64, F, P, P, L64, P, P, I, I, I, I, P, I, P]
+    lib.b200h_gated_conv.argtypes = [C.POINTER(RgLruArgs)]
+    lib.b200h_real_gated_scan.argtypes = [C.POINTER(RgLruArgs)]
+    lib.b200h_silu_mul_rows.argtypes = [P, I, I, P, I, P]
     _lib = lib
     return lib
 

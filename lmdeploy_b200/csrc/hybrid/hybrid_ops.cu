@@ -1,7 +1,8 @@
 // Operators of hybrid decoders (latent attention with a sink, decayed linear attention, routed experts, grouped RMS norm,
 // short causal convolution, depth-weighted residual history; window_attention.cuh: pre-norm blocks and windowed attention;
-// ssm.cuh, parallel_block.cuh: the state-space mixer, parallel blocks and convolved rotary attention) behind a C ABI of
-// their own: libb200hybrid.so.
+// ssm.cuh, parallel_block.cuh: the state-space mixer, parallel blocks and convolved rotary attention; token_shift.cuh: shared-norm
+// blocks and the channel-decay recurrence; gated_recurrence.cuh, normed_block.cuh: token-gated recurrences and blocks that norm a
+// sublayer's output) behind a C ABI of their own: libb200hybrid.so.
 //
 // Number formats.  T is the activation / weight type of the matrix products (float or bf16).  Everything the designs want in
 // 32 bits is float here whatever T is: the residual stream and its history, every norm, rotary angles (double), attention
@@ -460,11 +461,12 @@ __global__ void gated_rms_kernel(const float* __restrict__ o, const float* __res
 }
 
 // ------------------------------------------------------------------------------------------------ routed experts
-// Router: logits = router x (float); scores = softmax over all experts (score_fn 0) or the sigmoid of every logit on its own
-// (score_fn 1); the `top` largest (ties: the lower index), their scores as weights.  x is float or T.
+// Router: logits = router x + bias (float; bias nullptr: none); scores = softmax over all experts (score_fn 0), the sigmoid of every
+// logit on its own (score_fn 1) or softmax over the chosen logits only (score_fn 2); the `top` largest (ties: the lower index), their
+// scores as weights.  x is float or T.
 template <typename TI>
-__global__ void route_kernel(const TI* __restrict__ x, const float* __restrict__ router, int width, int experts, int top, int score_fn,
-                             int* __restrict__ ids, float* __restrict__ wts)
+__global__ void route_kernel(const TI* __restrict__ x, const float* __restrict__ router, const float* __restrict__ bias, int width, int experts,
+                             int top, int score_fn, int* __restrict__ ids, float* __restrict__ wts)
 {
     extern __shared__ float sm[];
     float* xs = sm;
@@ -477,13 +479,13 @@ __global__ void route_kernel(const TI* __restrict__ x, const float* __restrict__
         float part = 0.f;
         for (int i = lane; i < width; i += 32) part = fmaf(row[i], xs[i], part);
         part = warp_sum(part);
-        if (lane == 0) z[e] = part;
+        if (lane == 0) z[e] = part + (bias ? bias[e] : 0.f);
     }
     __syncthreads();
     if (threadIdx.x == 0) {
         float inv = 1.0f;
-        if (score_fn == 1) {
-            // the sigmoid is monotonic: the choice is made on the logits themselves (two large logits whose sigmoids both round
+        if (score_fn != 0) {
+            // the sigmoid and the softmax over the chosen are monotonic: the choice is made on the logits themselves (two large logits whose sigmoids both round
             // to one are still told apart), and only the chosen ones' sigmoids are taken
             for (int k = 0; k < top; ++k) {
                 int best = -1;
@@ -491,8 +493,18 @@ __global__ void route_kernel(const TI* __restrict__ x, const float* __restrict__
                 for (int e = 0; e < experts; ++e)
                     if (z[e] > bv || best < 0) { bv = z[e]; best = e; }
                 ids[(size_t)t * top + k] = best;
-                wts[(size_t)t * top + k] = sigmoid_f(bv);
+                wts[(size_t)t * top + k] = score_fn == 1 ? sigmoid_f(bv) : bv;
                 z[best] = -INFINITY;
+            }
+            if (score_fn == 2) {                              // the first choice has the largest logit
+                const float mx = wts[(size_t)t * top];
+                float sum = 0.f;
+                for (int k = 0; k < top; ++k) {
+                    const float e = expf(wts[(size_t)t * top + k] - mx);
+                    wts[(size_t)t * top + k] = e;
+                    sum += e;
+                }
+                for (int k = 0; k < top; ++k) wts[(size_t)t * top + k] /= sum;
             }
             return;
         } else {
@@ -784,6 +796,8 @@ __global__ void argmax_kernel(const float* __restrict__ logits, int64_t ld, int 
 #include "ssm.cuh"
 #include "parallel_block.cuh"
 #include "token_shift.cuh"
+#include "gated_recurrence.cuh"
+#include "normed_block.cuh"
 
 }  // namespace b200h
 
@@ -999,31 +1013,32 @@ B200H_API int b200h_gated_rms(const void* o, const void* w, const void* gate, in
 }
 
 template <typename TI>
-static void launch_route(const void* x, const void* router, int n, int width, int experts, int top, int score_fn, void* ids, void* wts,
-                         size_t smem, cudaStream_t st)
+static void launch_route(const void* x, const void* router, const void* bias, int n, int width, int experts, int top, int score_fn, void* ids,
+                         void* wts, size_t smem, cudaStream_t st)
 {
     if (smem > 48 * 1024) cudaFuncSetAttribute(route_kernel<TI>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    route_kernel<TI><<<n, 256, smem, st>>>((const TI*)x, (const float*)router, width, experts, top, score_fn, (int*)ids, (float*)wts);
+    route_kernel<TI><<<n, 256, smem, st>>>((const TI*)x, (const float*)router, (const float*)bias, width, experts, top, score_fn, (int*)ids,
+                                            (float*)wts);
 }
 
-B200H_API int b200h_route_scored(const void* x, int x_dtype, const void* router, int n, int width, int experts, int top, int score_fn,
-                                 void* ids, void* wts, void* stream)
+B200H_API int b200h_route_scored(const void* x, int x_dtype, const void* router, const void* bias, int n, int width, int experts, int top,
+                                 int score_fn, void* ids, void* wts, void* stream)
 {
-    if (!x || !router || !ids || !wts || experts <= 0 || top <= 0 || top > experts || score_fn < 0 || score_fn > 1)
+    if (!x || !router || !ids || !wts || experts <= 0 || top <= 0 || top > experts || score_fn < 0 || score_fn > 2)
         return fail(B200H_ERR_INVALID_ARG, "route: bad arguments");
     if (n == 0) return 0;
     const size_t smem = (size_t)(width + experts) * sizeof(float);
     if (smem > 200 * 1024) return fail(B200H_ERR_UNSUPPORTED, "route: width + experts exceeds shared memory");
     cudaStream_t st = (cudaStream_t)stream;
-    if (x_dtype == B200H_F32) launch_route<float>(x, router, n, width, experts, top, score_fn, ids, wts, smem, st);
-    else if (x_dtype == B200H_BF16) launch_route<bf16>(x, router, n, width, experts, top, score_fn, ids, wts, smem, st);
+    if (x_dtype == B200H_F32) launch_route<float>(x, router, bias, n, width, experts, top, score_fn, ids, wts, smem, st);
+    else if (x_dtype == B200H_BF16) launch_route<bf16>(x, router, bias, n, width, experts, top, score_fn, ids, wts, smem, st);
     else return fail(B200H_ERR_UNSUPPORTED, "dtype: float32 (2) or bfloat16 (1)");
     return launched("route");
 }
 
 B200H_API int b200h_route(const void* x, const void* router, int n, int width, int experts, int top, void* ids, void* wts, void* stream)
 {
-    return b200h_route_scored(x, B200H_F32, router, n, width, experts, top, 0, ids, wts, stream);
+    return b200h_route_scored(x, B200H_F32, router, nullptr, n, width, experts, top, 0, ids, wts, stream);
 }
 
 template <typename T>
@@ -1142,7 +1157,7 @@ static int window_args_ok(const b200h_window_args* a, const char** why)
 {
     if (!a || !a->tok_seq || !a->tok_pos || !a->block_ptrs || !a->cu_blocks || !a->qn) { *why = "window attention: bad arguments"; return 0; }
     if (a->heads <= 0 || a->kv_heads <= 0 || a->heads % a->kv_heads || a->dim <= 0 || a->vdim <= 0 || a->block_len <= 0 || a->window < 0 ||
-        a->chunk < 0 || (a->talk_scores && !a->talk)) {
+        a->chunk < 0 || (a->talk_scores && !a->talk) || !(a->q_temp_every >= 0.0)) {
         *why = "window attention: heads must be a multiple of kv_heads, sizes positive";
         return 0;
     }
@@ -1159,7 +1174,8 @@ B200H_API int b200h_window_prep(const b200h_window_args* a)
     B200H_DISPATCH_T(a->dtype, window_prep_kernel<T><<<a->n, 256, 0, st>>>(
         (const T*)a->q, (const T*)a->k, (const T*)a->v, a->ld, a->heads * a->dim, a->kv_heads * a->dim, a->kv_heads * a->vdim,
         (const float*)a->bias, (const float*)a->q_norm, (const float*)a->k_norm, a->eps, (const int*)a->tok_seq, (const int*)a->tok_pos,
-        (const int64_t*)a->block_ptrs, (const int*)a->cu_blocks, a->layer_off, a->v_off, a->block_len, (float*)a->qn));
+        (const int64_t*)a->block_ptrs, (const int*)a->cu_blocks, a->layer_off, a->v_off, a->block_len, a->q_temp_coef, a->q_temp_every,
+        (float*)a->qn));
     return launched("window_prep");
 }
 
@@ -1179,7 +1195,8 @@ B200H_API int b200h_head_rope_prep(const b200h_window_args* a, const b200h_rotar
         head_rope_prep_kernel<T><<<a->n, 256, smem, st>>>(
             (const T*)a->q, (const T*)a->k, (const T*)a->v, a->ld, a->heads, a->kv_heads, a->dim, a->vdim, (const float*)a->bias,
             (const float*)a->q_norm, (const float*)a->k_norm, a->eps, rot, (const int*)a->tok_seq, (const int*)a->tok_pos,
-            (const int64_t*)a->block_ptrs, (const int*)a->cu_blocks, a->layer_off, a->v_off, a->block_len, (float*)a->qn);
+            (const int64_t*)a->block_ptrs, (const int*)a->cu_blocks, a->layer_off, a->v_off, a->block_len, a->q_temp_coef,
+            a->q_temp_every, (float*)a->qn);
     });
     return launched("head_rope_prep");
 }
@@ -1234,7 +1251,9 @@ static int launch_window_attention(const b200h_window_args* a, WindowGeom g, cud
     const int span = a->window > 0 && a->chunk > 0 ? (a->window < a->chunk ? a->window : a->chunk) : (a->window > 0 ? a->window : a->chunk);
     const int keys = span > 0 ? span + g.rows - 1 : 1 << 30, per = (keys + a->splits - 1) / a->splits;
     l.stats_threads = per <= 32 ? 32 : (per <= 64 ? 64 : 128);
-    l.stats_smem = (size_t)g.rows * rep * a->dim * sizeof(float) + (VEC ? (size_t)l.stats_threads * (a->dim * sizeof(T) + 16) : 0);
+    auto stats_smem = [&]() { return (size_t)g.rows * rep * a->dim * sizeof(float) + (VEC ? (size_t)l.stats_threads * (a->dim * sizeof(T) + 16) : 0); };
+    while (stats_smem() > 200 * 1024 && l.stats_threads > 32) l.stats_threads /= 2;           // wide heads: fewer key rows staged at a time
+    l.stats_smem = stats_smem();
     l.pv_smem = window_pv_smem(a, g.rows, g.tile);
     if (l.stats_smem > 200 * 1024 || l.pv_smem > 200 * 1024)
         return fail(B200H_ERR_UNSUPPORTED, "window_attention: heads * (dim + vdim + heads) floats exceed an SM's shared memory");
@@ -1471,8 +1490,8 @@ B200H_API int b200h_channel_decay_scan(const void* r, const void* k, const void*
     const int groups = (vdim + 31) / 32, kw = (dim + 15) / 16;
     const dim3 grid(heads * groups, batch), block(32, kw);
     const size_t smem = (size_t)kw * (3 * 4 * 16 + 2 * 4 * 32) * sizeof(float);
-    B200H_DISPATCH_T(dtype, (channel_decay_scan_kernel<T, 4><<<grid, block, smem, st>>>(
-        (const T*)r, (const T*)k, (const T*)v, ld, (const float*)decay, (const float*)bonus, (float*)state, slot_stride, (const int*)cu_q,
+    B200H_DISPATCH_T(dtype, (channel_decay_scan_kernel<T, 4, false><<<grid, block, smem, st>>>(
+        (const T*)r, (const T*)k, (const T*)v, ld, 1.0f, (const float*)decay, (const float*)bonus, (float*)state, slot_stride, (const int*)cu_q,
         (const int*)seq_slot, heads, dim, vdim, (float*)out)));
     return launched("channel_decay_scan");
 }
@@ -1541,4 +1560,138 @@ B200H_API int b200h_route_grouped(const void* x, int x_dtype, const void* router
         launch_route_grouped<bf16>(x, router, correction, n, width, experts, top, groups, keep, group_top, renorm, scale, ids, wts, smem, st);
     else return fail(B200H_ERR_UNSUPPORTED, "dtype: float32 (2) or bfloat16 (1)");
     return launched("route_grouped");
+}
+
+// ------------------------------------------------------------------------------------------------ blocks with a norm on both ends of a sublayer
+B200H_API int b200h_normed_residual_norm(void* x, const void* left, const void* right, const void* wl, const void* wr, float branch_scale,
+                                         const void* m, const void* ff, int parts, const void* w_post, const void* w_next, int n, int width,
+                                         float eps, void* h, void* hf, int dtype, void* stream)
+{
+    if (!x || n < 0 || width <= 0 || (!left != !right) || (left && (!wl || !wr)) || (ff && parts < 1) || ((left || m || ff) && !w_post) ||
+        ((h || hf) && !w_next))
+        return fail(B200H_ERR_INVALID_ARG, "normed_residual_norm: bad arguments");
+    const size_t smem = (size_t)width * sizeof(float) * (left ? 2 : 1);
+    if (smem > 200 * 1024) return fail(B200H_ERR_UNSUPPORTED, "normed_residual_norm: a row exceeds shared memory");
+    if (n == 0) return 0;
+    cudaStream_t st = (cudaStream_t)stream;
+    const void* rows[] = {x, left, right, wl, wr, m, ff, w_post, w_next, h, hf};
+    bool vec = width % 4 == 0;
+    for (const void* p : rows) vec = vec && (reinterpret_cast<uintptr_t>(p) & 15) == 0;
+#define B200H_JOIN(V)                                                                                                                        \
+    do {                                                                                                                                    \
+        if (smem > 48 * 1024)                                                                                                               \
+            cudaFuncSetAttribute(normed_residual_norm_kernel<T, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                \
+        normed_residual_norm_kernel<T, V><<<n, 256, smem, st>>>((float*)x, (const T*)left, (const T*)right, (const float*)wl,               \
+            (const float*)wr, branch_scale, (const T*)m, (const float*)ff, ff ? parts : 0, (const float*)w_post, (const float*)w_next,      \
+            width, eps, (T*)h, (float*)hf);                                                                                                 \
+    } while (0)
+    B200H_DISPATCH_T(dtype, if (vec) B200H_JOIN(4); else B200H_JOIN(1));
+#undef B200H_JOIN
+    return launched("normed_residual_norm");
+}
+
+B200H_API int b200h_silu_mul_rows(const void* gu, int n, int cols, void* out, int dtype, void* stream)
+{
+    if (!gu || !out || n < 0 || cols <= 0) return fail(B200H_ERR_INVALID_ARG, "silu_mul_rows: bad arguments");
+    if (n == 0) return 0;
+    cudaStream_t st = (cudaStream_t)stream;
+    const int64_t count = (int64_t)n * cols;
+    if (cols % 4 == 0 && ((reinterpret_cast<uintptr_t>(gu) | reinterpret_cast<uintptr_t>(out)) & 15) == 0) {
+        B200H_DISPATCH_T(dtype, (silu_mul_rows_kernel<T, 4><<<(unsigned)((count / 4 + 255) / 256), 256, 0, st>>>((const T*)gu, cols, count, (T*)out)));
+    } else {
+        B200H_DISPATCH_T(dtype, (silu_mul_rows_kernel<T, 1><<<(unsigned)((count + 255) / 256), 256, 0, st>>>((const T*)gu, cols, count, (T*)out)));
+    }
+    return launched("silu_mul_rows");
+}
+
+// ------------------------------------------------------------------------------------------------ recurrences with token-dependent gates
+B200H_API int b200h_low_rank_decay(const void* low, int64_t ld, const void* a, const void* bias, int n, int channels, int rank, float tau,
+                                   void* decay, int dtype, void* stream)
+{
+    if (!low || !a || !bias || !decay || n < 0 || channels <= 0 || rank <= 0 || !(tau > 0.f))
+        return fail(B200H_ERR_INVALID_ARG, "low_rank_decay: bad arguments");
+    if (rank > 1024) return fail(B200H_ERR_UNSUPPORTED, "low_rank_decay: rank <= 1024");
+    if (n == 0) return 0;
+    cudaStream_t st = (cudaStream_t)stream;
+    const int cb = (channels + 255) / 256;
+    // eight rows share a read of `a`; one where that would leave SMs without a block
+#define B200H_LRD(ROWS)                                                                                                               \
+    low_rank_decay_kernel<T, ROWS><<<dim3(cb, (n + ROWS - 1) / ROWS), 256, (size_t)rank * ROWS * sizeof(float), st>>>(                 \
+        (const T*)low, ld, (const T*)a, (const float*)bias, n, channels, rank, 1.0f / tau, (float*)decay)
+    B200H_DISPATCH_T(dtype, if ((int64_t)cb * n >= 4096) B200H_LRD(8); else B200H_LRD(1));
+#undef B200H_LRD
+    return launched("low_rank_decay");
+}
+
+B200H_API int b200h_gated_linear_scan(const void* q, const void* k, const void* v, int64_t ld, float q_scale, const void* decay, void* state,
+                                      int64_t slot_stride, const void* cu_q, const void* seq_slot, int batch, int heads, int dim, int vdim,
+                                      void* out, int dtype, void* stream)
+{
+    if (!q || !k || !v || !decay || !state || !cu_q || !seq_slot || !out || batch <= 0 || heads <= 0 || dim <= 0 || vdim <= 0)
+        return fail(B200H_ERR_INVALID_ARG, "gated_linear_scan: bad arguments");
+    if (dim > 256) return fail(B200H_ERR_UNSUPPORTED, "gated_linear_scan: dim <= 256");
+    cudaStream_t st = (cudaStream_t)stream;
+    const int groups = (vdim + 31) / 32, kw = (dim + 15) / 16;
+    const dim3 grid(heads * groups, batch), block(32, kw);
+    const size_t smem = (size_t)kw * (3 * 4 * 16 + 2 * 4 * 32) * sizeof(float);
+    B200H_DISPATCH_T(dtype, (channel_decay_scan_kernel<T, 4, true><<<grid, block, smem, st>>>(
+        (const T*)q, (const T*)k, (const T*)v, ld, q_scale, (const float*)decay, nullptr, (float*)state, slot_stride, (const int*)cu_q,
+        (const int*)seq_slot, heads, dim, vdim, (float*)out)));
+    return launched("gated_linear_scan");
+}
+
+static bool rglru_args_ok(const b200h_rglru_args* a)
+{
+    return a && a->x && a->y && a->conv && a->conv_state && a->state && a->tok_seq && a->cu_q && a->seq_slot && a->u && a->n >= 0 && a->batch > 0 &&
+           a->width > 0 && a->blocks > 0 && a->width % a->blocks == 0 && a->ld >= a->width;
+}
+
+template <typename T>
+static void launch_gated_conv(const b200h_rglru_args* a, cudaStream_t st)
+{
+    const bool vec = a->width % 2 == 0 && a->ld % 2 == 0 && (reinterpret_cast<uintptr_t>(a->x) % (2 * sizeof(T))) == 0 &&
+                     (reinterpret_cast<uintptr_t>(a->u) % (2 * sizeof(T))) == 0;
+    const int v = vec ? 2 : 1, cb = ((a->width + v - 1) / v + 127) / 128;
+    const bool many = (int64_t)cb * a->n >= 8 * 1184;         // eight rows per block once that leaves eight blocks per SM
+#define B200H_CONV(TAPS, ROWS, V)                                                                                                           \
+    gated_conv_kernel<T, TAPS, ROWS, V><<<dim3(cb, (a->n + ROWS - 1) / ROWS), 128, 0, st>>>(                                                \
+        (const T*)a->x, a->ld, (const float*)a->x_bias, (const float*)a->conv, (const float*)a->conv_bias, a->taps, (const float*)a->conv_state, \
+        a->slot_stride, (const int*)a->tok_seq, (const int*)a->cu_q, (const int*)a->seq_slot, a->n, a->width, (T*)a->u)
+#define B200H_CONV_V(TAPS, ROWS) do { if (vec) B200H_CONV(TAPS, ROWS, 2); else B200H_CONV(TAPS, ROWS, 1); } while (0)
+    if (a->taps <= 4) { if (many) B200H_CONV_V(4, 8); else B200H_CONV_V(4, 1); }
+    else B200H_CONV_V(B200H_MAX_TAPS, 1);
+#undef B200H_CONV_V
+#undef B200H_CONV
+}
+
+B200H_API int b200h_gated_conv(const b200h_rglru_args* a)
+{
+    if (!rglru_args_ok(a)) return fail(B200H_ERR_INVALID_ARG, "gated_conv: bad arguments");
+    if (a->taps < 1 || a->taps > B200H_MAX_TAPS) return fail(B200H_ERR_UNSUPPORTED, "gated_conv: taps 1..16");
+    if (a->n == 0) return 0;
+    cudaStream_t st = (cudaStream_t)a->stream;
+    B200H_DISPATCH_T(a->dtype, launch_gated_conv<T>(a, st));
+    return launched("gated_conv");
+}
+
+B200H_API int b200h_real_gated_scan(const b200h_rglru_args* a)
+{
+    if (!rglru_args_ok(a) || !a->z || !a->lam || !a->out) return fail(B200H_ERR_INVALID_ARG, "real_gated_scan: bad arguments");
+    if (a->taps < 1 || a->taps > B200H_MAX_TAPS) return fail(B200H_ERR_UNSUPPORTED, "real_gated_scan: taps 1..16");
+    if (a->n == 0) return 0;
+    cudaStream_t st = (cudaStream_t)a->stream;
+    GatedScan g;
+    g.z = (const float*)a->z; g.r_bias = (const float*)a->r_bias; g.i_bias = (const float*)a->i_bias; g.lam = (const float*)a->lam;
+    g.state = (float*)a->state; g.slot_stride = a->slot_stride; g.cu_q = (const int*)a->cu_q; g.seq_slot = (const int*)a->seq_slot;
+    g.n = a->n; g.width = a->width; g.bw = a->width / a->blocks; g.taps = a->taps; g.rate = a->rate; g.ld = a->ld;
+    g.x_bias = (const float*)a->x_bias; g.y_bias = (const float*)a->y_bias; g.conv_state = (float*)a->conv_state;
+    // single rows: a thread per channel; portions: sixteen row groups of eight rows per tile
+    if (a->n == a->batch) {
+        B200H_DISPATCH_T(a->dtype, (real_gated_scan_kernel<T, 1><<<dim3((a->width + 127) / 128, a->batch), dim3(128, 1), 0, st>>>(
+            g, (const T*)a->x, (const T*)a->y, (const T*)a->u, (T*)a->out)));
+    } else {
+        B200H_DISPATCH_T(a->dtype, (real_gated_scan_kernel<T, 8><<<dim3((a->width + 31) / 32, a->batch), dim3(32, 16), 2 * 2 * 16 * 32 * sizeof(float), st>>>(
+            g, (const T*)a->x, (const T*)a->y, (const T*)a->u, (T*)a->out)));
+    }
+    return launched("real_gated_scan");
 }

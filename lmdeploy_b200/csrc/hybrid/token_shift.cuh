@@ -140,7 +140,9 @@ __global__ void channel_decay_kernel(const float* __restrict__ d, const float* _
     if (i < count) decay[i] = expf(-expf(d[i] + w0[i % channels]));
 }
 
-// Per head, with S a [dim, vdim] float matrix per sequence:  o_t = (S + diag(u) k_t v_t^T)^T r_t,  S <- diag(w_t) S + k_t v_t^T.
+// Per head, with S a [dim, vdim] float matrix per sequence and the row's r scaled by r_scale:
+//   AFTER false:  o_t = (S + diag(u) k_t v_t^T)^T r_t,  S <- diag(w_t) S + k_t v_t^T    (the state is read before the row joins it)
+//   AFTER true:   S <- diag(w_t) S + k_t v_t^T,  o_t = S^T r_t                          (after; no bonus term)
 // One block owns 32 value columns of one (sequence, head); its warps split the key channels, 16 each: lane j of warp w keeps
 // S[16 w .. 16 w + 15, j] in registers, so a row costs no shuffle per column.  With c = sum_i r_i u_i k_i (the bonus term, common to
 // all columns) a warp's part of a row is  sum_(its i) r_i S_ij + v_j c_(its i);  then S_ij <- w_i S_ij + k_i v_j.  The parts of R
@@ -149,9 +151,9 @@ __global__ void channel_decay_kernel(const float* __restrict__ d, const float* _
 // broadcasts); the next R rows' global loads are in flight while the current ones are computed.
 // r, k, v: T with row stride ld; decay: float [n, heads * dim].  State layout per head: [vdim][dim] floats.
 // blockDim = (32, ceil(dim / 16)); grid = (heads * ceil(vdim / 32), batch).  Channels past dim hold zeros and stay zero.
-template <typename T, int R>
+template <typename T, int R, bool AFTER>
 __global__ void __launch_bounds__(512) channel_decay_scan_kernel(const T* __restrict__ r, const T* __restrict__ k, const T* __restrict__ v,
-                                                                int64_t ld, const float* __restrict__ decay, const float* __restrict__ bonus,
+                                                                int64_t ld, float r_scale, const float* __restrict__ decay, const float* __restrict__ bonus,
                                                                 float* __restrict__ state, int64_t slot_stride, const int* __restrict__ cu_q,
                                                                 const int* __restrict__ seq_slot, int heads, int dim, int vdim,
                                                                 float* __restrict__ out)
@@ -184,7 +186,7 @@ __global__ void __launch_bounds__(512) channel_decay_scan_kernel(const T* __rest
     // staged element e of a lane: row (e * 32 + lane) / CK of the group, the warp's channel (e * 32 + lane) % CK
     const int my_d = c0 + lane % CK, my_u = lane / CK;
     const bool my_in = my_d < dim;
-    const float ub = my_in ? bonus[(size_t)h * dim + my_d] : 0.f;
+    const float ub = !AFTER && my_in ? bonus[(size_t)h * dim + my_d] : 0.f;
     const size_t hd = (size_t)heads * dim, my_at = (size_t)h * dim + my_d;
     float rr[E], kk[E], ww[E], vv[R];
     // the loads of rows [t0, t0 + R) into registers (zeros past the sequence's last row and past dim)
@@ -207,14 +209,16 @@ __global__ void __launch_bounds__(512) channel_decay_scan_kernel(const T* __rest
 #pragma unroll
         for (int e = 0; e < E; ++e) {
             const int at = e * 32 + lane;                    // = row * CK + channel
-            rs[at] = rr[e];
+            rs[at] = rr[e] * r_scale;
             ks[at] = kk[e];
             wd[at] = ww[e];
-            float c = rr[e] * ub * kk[e];                    // the bonus term of this warp's channels: summed over the CK lanes of a row
+            if (!AFTER) {
+                float c = rs[at] * ub * kk[e];               // the bonus term of this warp's channels: summed over the CK lanes of a row
 #pragma unroll
-            for (int o = CK / 2; o > 0; o >>= 1) c += __shfl_xor_sync(0xffffffffu, c, o);
+                for (int o = CK / 2; o > 0; o >>= 1) c += __shfl_xor_sync(0xffffffffu, c, o);
 #pragma unroll
-            for (int q = 0; q < 32 / CK; ++q) cc[e * (32 / CK) + q] = __shfl_sync(0xffffffffu, c, q * CK);
+                for (int q = 0; q < 32 / CK; ++q) cc[e * (32 / CK) + q] = __shfl_sync(0xffffffffu, c, q * CK);
+            }
         }
 #pragma unroll
         for (int u = 0; u < R; ++u) vc[u] = vv[u];
@@ -231,12 +235,19 @@ __global__ void __launch_bounds__(512) channel_decay_scan_kernel(const T* __rest
                     const float4 r4 = *reinterpret_cast<const float4*>(rs + u * CK + i);
                     const float4 k4 = *reinterpret_cast<const float4*>(ks + u * CK + i);
                     const float4 w4 = *reinterpret_cast<const float4*>(wd + u * CK + i);
-                    a0 = fmaf(r4.x, S[i], a0);     S[i] = fmaf(w4.x, S[i], k4.x * vj);
-                    a1 = fmaf(r4.y, S[i + 1], a1); S[i + 1] = fmaf(w4.y, S[i + 1], k4.y * vj);
-                    a2 = fmaf(r4.z, S[i + 2], a2); S[i + 2] = fmaf(w4.z, S[i + 2], k4.z * vj);
-                    a3 = fmaf(r4.w, S[i + 3], a3); S[i + 3] = fmaf(w4.w, S[i + 3], k4.w * vj);
+                    if (AFTER) {
+                        S[i] = fmaf(w4.x, S[i], k4.x * vj);         a0 = fmaf(r4.x, S[i], a0);
+                        S[i + 1] = fmaf(w4.y, S[i + 1], k4.y * vj); a1 = fmaf(r4.y, S[i + 1], a1);
+                        S[i + 2] = fmaf(w4.z, S[i + 2], k4.z * vj); a2 = fmaf(r4.z, S[i + 2], a2);
+                        S[i + 3] = fmaf(w4.w, S[i + 3], k4.w * vj); a3 = fmaf(r4.w, S[i + 3], a3);
+                    } else {
+                        a0 = fmaf(r4.x, S[i], a0);     S[i] = fmaf(w4.x, S[i], k4.x * vj);
+                        a1 = fmaf(r4.y, S[i + 1], a1); S[i + 1] = fmaf(w4.y, S[i + 1], k4.y * vj);
+                        a2 = fmaf(r4.z, S[i + 2], a2); S[i + 2] = fmaf(w4.z, S[i + 2], k4.z * vj);
+                        a3 = fmaf(r4.w, S[i + 3], a3); S[i + 3] = fmaf(w4.w, S[i + 3], k4.w * vj);
+                    }
                 }
-                mine[u * 32] = fmaf(vj, cc[u], (a0 + a1) + (a2 + a3));
+                mine[u * 32] = AFTER ? (a0 + a1) + (a2 + a3) : fmaf(vj, cc[u], (a0 + a1) + (a2 + a3));
             }
         }
         __syncthreads();

@@ -64,15 +64,22 @@ __global__ void relu2_kernel(T* __restrict__ x, int64_t count)
     x[i] = from_f<T>(v * v);
 }
 
+// The factor on a query at position pos: 1 + coef * ln(1 + floor((pos + 1) / every)); every 0: one.  (The quotient in double: exact at
+// the multiples of `every`, and never rounded up to one.)
+__device__ __forceinline__ float query_growth(int pos, float coef, double every)
+{
+    return every > 0.0 ? fmaf(coef, logf((float)floor((double)(pos + 1) / every) + 1.0f), 1.0f) : 1.0f;
+}
+
 // One block per row: the projections' biases are added (float), the query is normed over all its heads at once (-> qn, float), the
 // key likewise and written to the row's cache entry as T, the value is written to the cache.  wq / wk == nullptr: no norm of that
-// projection; bias (q | k | v entries, float) == nullptr: none.
+// projection; the query grows with its position (query_growth); bias (q | k | v entries, float) == nullptr: none.
 template <typename T>
 __global__ void window_prep_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __restrict__ v, int64_t ld, int q_cols,
                                    int k_cols, int v_cols, const float* __restrict__ bias, const float* __restrict__ wq,
                                    const float* __restrict__ wk, float eps, const int* __restrict__ tok_seq, const int* __restrict__ tok_pos,
                                    const int64_t* __restrict__ block_ptrs, const int* __restrict__ cu_blocks, int64_t layer_off, int64_t v_off,
-                                   int block_len, float* __restrict__ qn)
+                                   int block_len, float q_temp_coef, double q_temp_every, float* __restrict__ qn)
 {
     __shared__ float red[32];
     const int t = blockIdx.x, s = tok_seq[t], pos = tok_pos[t];
@@ -80,6 +87,7 @@ __global__ void window_prep_kernel(const T* __restrict__ q, const T* __restrict_
     const float* bk = bias ? bias + q_cols : nullptr;
     const float* bv = bias ? bias + q_cols + k_cols : nullptr;
     const T* qr = q + (size_t)t * ld;
+    const float growth = query_growth(pos, q_temp_coef, q_temp_every);
     float r = 1.0f;
     if (wq) {
         float ss = 0.f;
@@ -89,7 +97,7 @@ __global__ void window_prep_kernel(const T* __restrict__ q, const T* __restrict_
     }
     for (int i = threadIdx.x; i < q_cols; i += blockDim.x) {
         const float a = to_f(qr[i]) + (bq ? bq[i] : 0.f);
-        qn[(size_t)t * q_cols + i] = wq ? a * r * wq[i] : a;
+        qn[(size_t)t * q_cols + i] = (wq ? a * r * wq[i] : a) * growth;
     }
     char* page = reinterpret_cast<char*>(block_ptrs[cu_blocks[s] + pos / block_len]) + layer_off;
     const int at = pos % block_len;
@@ -519,7 +527,7 @@ __global__ void __launch_bounds__(256) window_mix_scores_kernel(WindowGeom g, co
 //   2. every head of q and of k is divided by its root mean square over `dim` and multiplied by a weight of `dim` entries that all
 //      heads share (wq / wk; nullptr: no norm of that projection);
 //   3. pairs (2i, 2i+1), i < rot.pairs, of every head turn by position * freqs[i];
-//   4. queries -> qn (float), keys and (biased) values -> the row's cache entry as T.
+//   4. queries, times query_growth -> qn (float), keys and (biased) values -> the row's cache entry as T.
 // Shared memory: (heads + kv_heads) * dim floats, then 2 * rot.pairs floats of cos / sin.
 template <typename T>
 __global__ void head_rope_prep_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __restrict__ v, int64_t ld, int heads,
@@ -527,11 +535,12 @@ __global__ void head_rope_prep_kernel(const T* __restrict__ q, const T* __restri
                                       const float* __restrict__ wk, float eps, Rotary rot, const int* __restrict__ tok_seq,
                                       const int* __restrict__ tok_pos, const int64_t* __restrict__ block_ptrs,
                                       const int* __restrict__ cu_blocks, int64_t layer_off, int64_t v_off, int block_len,
-                                      float* __restrict__ qn)
+                                      float q_temp_coef, double q_temp_every, float* __restrict__ qn)
 {
     extern __shared__ __align__(16) float hr_smem[];
     const int t = blockIdx.x, s = tok_seq[t], pos = tok_pos[t];
     const int HD = heads * dim, GD = kv_heads * dim, GV = kv_heads * vdim;
+    const float growth = query_growth(pos, q_temp_coef, q_temp_every);
     float* buf = hr_smem;
     float* cs = hr_smem + HD + GD;
     float* sn = cs + rot.pairs;
@@ -573,8 +582,8 @@ __global__ void head_rope_prep_kernel(const T* __restrict__ q, const T* __restri
                 b = rb;
             }
             if (h < heads) {
-                qn[(size_t)t * HD + (size_t)h * dim + d] = a;
-                if (two) qn[(size_t)t * HD + (size_t)h * dim + d + 1] = b;
+                qn[(size_t)t * HD + (size_t)h * dim + d] = a * growth;
+                if (two) qn[(size_t)t * HD + (size_t)h * dim + d + 1] = b * growth;
             } else {
                 k_dst[(size_t)(h - heads) * dim + d] = from_f<T>(a);
                 if (two) k_dst[(size_t)(h - heads) * dim + d + 1] = from_f<T>(b);

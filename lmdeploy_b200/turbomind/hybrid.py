@@ -6,8 +6,9 @@ A hybrid decoder mixes layer kinds, so a sequence owns two things between steps:
     windowed-, chunked- or convolved-rotary-attention layer its normed (and rotated) keys and its values (as T);
   * one slot of the StatePool (handed out by scheduler.Scheduler's slot list) -- per layer the last taps-1 inputs of the
     short convolution (of both sublayers in pre-norm blocks; of the stacked q | k projection of a convolved attention; of the
-    x | B | C channels of a state-space mixer), per decayed-linear-attention or channel-decay layer the [heads, vdim, dim] float
-    state and per state-space layer the [heads, vdim, state] float state; in shared-norm blocks per run the last normed row and the
+    x | B | C channels of a state-space mixer; of the biased convolution branch of an RG-LRU), per decayed-linear-attention,
+    channel-decay or gated-linear layer the [heads, vdim, dim] float state, per state-space layer the [heads, vdim, state] float
+    state and per RG-LRU one float per channel; in shared-norm blocks per run the last normed row and the
     last shifted row (the token shift), and once the id of the last token (hashed bigram embedding).
 A layer that a spec loops (HybridSpec.loop) is executed several times per step with the same weights: caches and states
 belong to RUNS (HybridSpec.runs()), weights to layers.
@@ -82,7 +83,7 @@ class HybridModel:
         self.cache_off, self.rot_off, self.conv_off, self.mix_off, self.conv2_off, self.v_off = {}, {}, {}, {}, {}, {}
         self.shift_off = {}
         self.runs = spec.runs()
-        if spec.block not in ("post_norm", "pre_norm", "parallel", "shared_norm"):
+        if spec.block not in ("post_norm", "pre_norm", "parallel", "shared_norm", "sandwich"):
             raise NotImplementedError(f"block {spec.block!r}")
         pre = spec.block == "pre_norm"
         page = slot = 0
@@ -98,7 +99,7 @@ class HybridModel:
             if spec.block == "shared_norm":     # token shift: the last normed row and the last shifted row
                 self.shift_off[r] = slot
                 slot += 2 * spec.width
-            elif spec.block != "parallel":
+            elif spec.block not in ("parallel", "sandwich"):
                 slot += (taps - 1) * spec.width
             if pre and layer.mlp is not None:
                 self.conv2_off[r] = slot
@@ -136,10 +137,11 @@ class HybridModel:
                 slot += m.heads * m.vdim * m.dim
             elif m.kind in ("window_attention", "paired"):
                 if m.kind == "paired":
-                    if spec.block != "shared_norm" or m.left.kind != "window_attention" or m.right.kind != "channel_decay":
-                        raise NotImplementedError("paired mixers: windowed attention beside a channel-decay recurrence in shared-norm blocks")
+                    if m.left.kind != "window_attention" or (spec.block, m.right.kind) not in (("shared_norm", "channel_decay"), ("sandwich", "gated_linear")):
+                        raise NotImplementedError("paired mixers: windowed attention beside a channel-decay recurrence in shared-norm blocks "
+                                                  "or beside gated linear attention in sandwich blocks")
                     if m.right.dim > 256:
-                        raise NotImplementedError("channel-decay recurrence: dim <= 256")
+                        raise NotImplementedError("channel-decay recurrence, gated linear attention: dim <= 256")
                     slot = _align(slot, 4)                  # 16-byte reads of the state's columns
                     self.mix_off[r] = slot
                     slot += m.right.heads * m.right.vdim * m.right.dim
@@ -150,6 +152,13 @@ class HybridModel:
                 self.cache_off[r] = page
                 self.v_off[r] = _align(block_len * m.kv_heads * m.dim * esize)
                 page += self.v_off[r] + _align(block_len * m.kv_heads * m.vdim * esize)
+            elif m.kind == "rglru":
+                if not 1 <= m.conv_taps <= H.MAX_TAPS:
+                    raise NotImplementedError(f"conv taps {m.conv_taps} (1..{H.MAX_TAPS})")
+                self.conv_off[r] = slot
+                slot += (m.conv_taps - 1) * m.width
+                self.mix_off[r] = slot
+                slot += m.width
             else:
                 raise NotImplementedError(m.kind)
         self.block_bytes = max(page, 16)
@@ -232,7 +241,7 @@ class HybridModel:
 
         w["embed"] = lin("embed", shape=(s.vocab, W))
         w["head"] = w["embed"] if s.tied_head else lin("head", shape=(s.vocab, W))
-        w["final.norm"] = norm_w("final.norm")
+        w["final.norm"] = norm_w("final.norm") * s.logit_scale          # the head is linear in it: scaling the norm scales the logits
         if s.bigram is not None:
             w["bigram"] = lin("bigram", shape=(s.bigram.buckets + 1, W))
         if s.max_positions:
@@ -242,9 +251,11 @@ class HybridModel:
         for i, layer in enumerate(s.layers):
             p, m = f"l{i}.", layer.mixer
             w[p + "norm1"] = norm_w(p + "norm1")
-            shared = s.block == "shared_norm"
+            shared, both_ends = s.block == "shared_norm", s.block == "sandwich"
             if shared:
                 w[p + "shift"] = f32(p + "shift", (W,))
+            elif both_ends:
+                w[p + "norm1b"] = norm_w(p + "norm1b")
             elif not par:
                 w[p + "canon1"] = f32(p + "canon1", (W, s.conv_taps))
             if s.block == "post_norm":
@@ -282,6 +293,31 @@ class HybridModel:
                 w[p + "mag"] = float(mag)
             elif m.kind == "window_attention":
                 window_weights(p, p + "mix.", m)
+            elif m.kind == "rglru":
+                R = m.width
+                size = R // m.blocks
+                w[p + "in"] = lin(p + "mix.y", p + "mix.x", shape=(2 * R, W))
+                for k in ("y.b", "x.b", "conv.b", "lam"):
+                    w[p + k] = f32(p + "mix." + k, (R,))
+                w[p + "conv"] = f32(p + "mix.conv", (R, m.conv_taps))
+                # a block's two square maps stacked: one batched product over the blocks gives both gates
+                w[p + "gates"] = torch.cat([lin(p + "mix.ra", shape=(m.blocks, size, size)), lin(p + "mix.ri", shape=(m.blocks, size, size))], 1).contiguous()
+                for k in ("ra.b", "ri.b"):
+                    w[p + k] = f32(p + "mix." + k, (m.blocks, size)).reshape(R)
+                w[p + "o"] = lin(p + "mix.o", shape=(W, R))
+            elif m.kind == "paired" and m.right.kind == "gated_linear":
+                window_weights(p + "left.", p + "mix.left.", m.left)
+                R, ck = m.right, p + "mix.right."
+                HD, HV = R.heads * R.dim, R.heads * R.vdim
+                # both sides read the same rows: ONE product for left q | k | v and right q | k | v | g | a1
+                right_in = lin(*(ck + k for k in ("q", "k", "v", "g", "a1")), shape=(2 * HD + 2 * HV + R.rank, W))
+                w[p + "in"] = torch.cat([w.pop(p + "left.in"), right_in]).contiguous()
+                w[p + "right.a2"] = lin(ck + "a2", shape=(HD, R.rank)).t().contiguous()
+                w[p + "right.a2.b"] = f32(ck + "a2.b", (HD,))
+                w[p + "right.norm"] = f32(ck + "norm", (R.vdim,)).repeat(R.heads)
+                w[p + "right.o"] = lin(ck + "o", shape=(W, HV))
+                w[p + "left.out"] = f32(p + "mix.left.out", (W,))
+                w[p + "right.out"] = f32(p + "mix.right.out", (W,))
             elif m.kind == "paired":
                 window_weights(p + "left.", p + "mix.left.", m.left)
                 R, ck = m.right, p + "mix.right."
@@ -307,15 +343,25 @@ class HybridModel:
             if f is not None:
                 if not shared:
                     w[p + "norm2"] = norm_w(p + "norm2")
+                if both_ends:
+                    w[p + "norm2b"] = norm_w(p + "norm2b")
                 if pre:
                     w[p + "canon2"] = f32(p + "canon2", (W, s.conv_taps))
                 if f.kind == "dense":
-                    w[p + "up"] = lin(p + "mlp.up", shape=(f.ff, W))
+                    if f.act == "silu_gate":
+                        w[p + "up"] = lin(p + "mlp.gate", p + "mlp.up", shape=(2 * f.ff, W))
+                    else:
+                        w[p + "up"] = lin(p + "mlp.up", shape=(f.ff, W))
                     w[p + "down"] = lin(p + "mlp.down", shape=(W, f.ff))
                     if f.act == "xielu":
                         w[p + "act"] = f32(p + "mlp.act", (2,))
                     continue
                 w[p + "router"] = f32(p + "mlp.router", (f.experts, W))
+                if f.router_bias:
+                    w[p + "router.b"] = f32(p + "mlp.router.b", (f.experts,))
+                if f.shared:
+                    w[p + "shared.up"] = lin(p + "mlp.shared.gate", p + "mlp.shared.up", shape=(2 * f.shared, W))
+                    w[p + "shared.down"] = lin(p + "mlp.shared.down", shape=(W, f.shared))
                 if f.correction:
                     w[p + "correction"] = f32(p + "mlp.correction", (f.experts,))
                 for part, shape in (("gate", (f.ff, W)), ("up", (f.ff, W)), ("down", (W, f.ff))):
@@ -342,7 +388,7 @@ class HybridModel:
                 return torch.log(torch.expm1(0.001 + 0.099 * torch.rand(shape, generator=g)))
             if name.endswith(".D"):
                 return torch.ones(shape)
-            if name.endswith(("norm1", "norm2", ".norm", ".out")):
+            if name.endswith(("norm1", "norm2", "norm1b", "norm2b", ".norm", ".out")):
                 return 1.0 + 0.1 * torch.randn(shape, generator=g)
             if name.endswith("shift") or ".mu." in name:
                 return torch.rand(shape, generator=g)
@@ -350,6 +396,8 @@ class HybridModel:
                 return -6.0 + 6.0 * torch.rand(shape, generator=g)
             if name.endswith(".u"):
                 return 0.5 * torch.randn(shape, generator=g)
+            if name.endswith(".lam"):                                    # a = exp(-8 r softplus(lam)) between about 0.9 and 0.999 at r = 1
+                return -9.0 + 4.0 * torch.rand(shape, generator=g)
             if name.endswith("mlp.act"):
                 return torch.tensor([0.5, -0.5])
             if name.endswith("correction"):
@@ -386,7 +434,7 @@ class HybridModel:
             out["pos"] = (s.max_positions, W)
         if s.loop is not None:
             out["loop.step"] = (s.loop[2], W)
-        shared = s.block == "shared_norm"
+        shared, both_ends = s.block == "shared_norm", s.block == "sandwich"
 
         def window_shapes(ck, m):
             HD, GD, GV, HV = m.heads * m.dim, m.kv_heads * m.dim, m.kv_heads * m.vdim, m.heads * m.vdim
@@ -409,6 +457,8 @@ class HybridModel:
             out[p + "norm1"] = (W,)
             if shared:
                 out[p + "shift"] = (W,)
+            elif both_ends:
+                out[p + "norm1b"] = (W,)
             elif not par:
                 out[p + "canon1"] = (W, s.conv_taps)
             if s.block == "post_norm":
@@ -429,6 +479,18 @@ class HybridModel:
                             p + "mix.g": (HV, W), p + "mix.o": (W, HV)})
             elif m.kind == "window_attention":
                 window_shapes(p + "mix.", m)
+            elif m.kind == "rglru":
+                R, size = m.width, m.width // m.blocks
+                out.update({p + "mix.y": (R, W), p + "mix.x": (R, W), p + "mix.conv": (R, m.conv_taps), p + "mix.o": (W, R)})
+                out.update({p + "mix." + k: (R,) for k in ("y.b", "x.b", "conv.b", "lam")})
+                for k in ("ra", "ri"):
+                    out.update({p + "mix." + k: (m.blocks, size, size), p + f"mix.{k}.b": (m.blocks, size)})
+            elif m.kind == "paired" and m.right.kind == "gated_linear":
+                window_shapes(p + "mix.left.", m.left)
+                R, ck = m.right, p + "mix.right."
+                HD, HV = R.heads * R.dim, R.heads * R.vdim
+                out.update({ck + "q": (HD, W), ck + "k": (HD, W), ck + "v": (HV, W), ck + "g": (HV, W), ck + "a1": (R.rank, W), ck + "a2": (HD, R.rank),
+                            ck + "a2.b": (HD,), ck + "norm": (R.vdim,), ck + "o": (W, HV), p + "mix.left.out": (W,), p + "mix.right.out": (W,)})
             elif m.kind == "paired":
                 window_shapes(p + "mix.left.", m.left)
                 R, ck = m.right, p + "mix.right."
@@ -445,14 +507,22 @@ class HybridModel:
             if f is not None:
                 if not shared:
                     out[p + "norm2"] = (W,)
+                if both_ends:
+                    out[p + "norm2b"] = (W,)
                 if pre:
                     out[p + "canon2"] = (W, s.conv_taps)
                 if f.kind == "dense":
+                    if f.act == "silu_gate":
+                        out[p + "mlp.gate"] = (f.ff, W)
                     out.update({p + "mlp.up": (f.ff, W), p + "mlp.down": (W, f.ff)})
                     if f.act == "xielu":
                         out[p + "mlp.act"] = (2,)
                     continue
                 out[p + "mlp.router"] = (f.experts, W)
+                if f.router_bias:
+                    out[p + "mlp.router.b"] = (f.experts,)
+                if f.shared:
+                    out.update({f"{p}mlp.shared.gate": (f.shared, W), f"{p}mlp.shared.up": (f.shared, W), f"{p}mlp.shared.down": (W, f.shared)})
                 if f.correction:
                     out[p + "mlp.correction"] = (f.experts,)
                 for e in range(f.experts):
@@ -500,6 +570,10 @@ class HybridModel:
         st = self._stream()
         if s.max_positions and max_pos >= s.max_positions:
             raise ValueError(f"position {max_pos}: the model has {s.max_positions} learned positions")
+        if s.block == "sandwich":
+            return self._step_sandwich(n=n, batch=batch, tokens=tokens, tok_seq=tok_seq, tok_pos=tok_pos, cu_q=cu_q, seq_slot=seq_slot,
+                                       block_ptrs=block_ptrs, cu_blocks=cu_blocks, state=state, rows=rows, n_rows=n_rows, max_pos=max_pos,
+                                       trace=trace)
         if s.block == "shared_norm":
             return self._step_shared_norm(n=n, batch=batch, tokens=tokens, tok_seq=tok_seq, tok_pos=tok_pos, cu_q=cu_q, seq_slot=seq_slot,
                                           block_ptrs=block_ptrs, cu_blocks=cu_blocks, state=state, rows=rows, n_rows=n_rows,
@@ -716,6 +790,129 @@ class HybridModel:
                                               dt, st), "group_norm_rows")
             return self._logits(xn)
 
+    def _step_sandwich(self, *, n, batch, tokens, tok_seq, tok_pos, cu_q, seq_slot, block_ptrs, cu_blocks, state, rows, n_rows, max_pos,
+                       trace=None):
+        """The step of sandwich blocks: x <- x + n1b(mixer(n1(x))), x <- x + n2b(ff(n2(x))) per run.  One kernel per sublayer takes the
+        previous sublayer's output (the two sides of a paired mixer, one row, or the chosen experts' parts beside the shared one's),
+        norms it, adds it to the float stream and emits the next sublayer's normed input."""
+        s, lib, w, dev, T, dt = self.spec, self.lib, self.w, self.device, self.T, self.dt
+        W, eps, st = s.width, s.norm_eps, self._stream()
+        c = StepArrays(n=n, batch=batch, tok_seq=tok_seq, tok_pos=tok_pos, cu_q=cu_q, seq_slot=seq_slot, block_ptrs=block_ptrs,
+                       cu_blocks=cu_blocks, state=state, max_pos=max_pos)
+        x = torch.empty(n, W, dtype=torch.float32, device=dev)
+        with self.timed("embed"):
+            H.check(lib.b200h_embed(tokens.data_ptr(), w["embed"].data_ptr(), s.embedding_scale, x.data_ptr(), n, W, dt, st), "embed")
+        h = torch.empty(n, W, dtype=T, device=dev)
+        hf = torch.empty(n, W, dtype=torch.float32, device=dev)          # the router reads the second norm unrounded
+        pending = {}                     # a sublayer's output that the stream has not taken in yet
+
+        def ptr(t):
+            return None if t is None else t.data_ptr()
+
+        def join(norm, router=False):
+            nonlocal pending
+            q = pending
+            ff = q.get("ff")
+            with self.timed("post-norm + residual + norm"):
+                H.check(lib.b200h_normed_residual_norm(
+                    x.data_ptr(), ptr(q.get("left")), ptr(q.get("right")), ptr(q.get("wl")), ptr(q.get("wr")), 0.5, ptr(q.get("row")), ptr(ff),
+                    0 if ff is None else ff.shape[1], ptr(q.get("norm")), ptr(norm), n, W, eps, None if norm is None else h.data_ptr(),
+                    hf.data_ptr() if router else None, dt, st), "normed_residual_norm")
+            pending = {}
+
+        for r, (i, _) in enumerate(self.runs):
+            p, layer = f"l{i}.", s.layers[i]
+            m, f = layer.mixer, layer.mlp
+            join(w[p + "norm1"])
+            if m.kind == "paired":
+                with self.timed("gemm in"):
+                    proj = self._linear(h, w[p + "in"])
+                L = m.left
+                cols = (L.heads + L.kv_heads) * L.dim + L.kv_heads * L.vdim
+                y = self.window_mixer(i, None, c, run=r, m=L, p=p + "left.", proj=proj[:, :cols])
+                with self.timed("gemm out"):
+                    left = self._linear(y, w[p + "left.o"])
+                y = self.gated_linear_mixer(i, proj[:, cols:], c, run=r, m=m.right, p=p + "right.")
+                with self.timed("gemm out"):
+                    right = self._linear(y, w[p + "right.o"])
+                pending = dict(left=left, right=right, wl=w[p + "left.out"], wr=w[p + "right.out"], norm=w[p + "norm1b"])
+            else:
+                y = self.mixer(r, i, h, c)
+                with self.timed("gemm out"):
+                    pending = dict(row=self._linear(y, w[p + "o"]), norm=w[p + "norm1b"])
+            if f is not None:
+                routed = f.kind == "moe"
+                join(w[p + "norm2"], routed)
+                if routed:
+                    row = self.gated_mlp(h, w[p + "shared.up"], w[p + "shared.down"], "shared expert") if f.shared else None
+                    pending = dict(row=row, ff=self.routed_experts(i, hf, h, n), norm=w[p + "norm2b"])
+                else:
+                    pending = dict(row=self.dense_mlp(i, h), norm=w[p + "norm2b"])
+            if trace is not None:
+                join(None)
+                trace.append(x.clone())
+        xn = torch.empty(n_rows, W, dtype=T, device=dev)
+        with self.timed("final norm + head"):
+            if pending:
+                join(None)
+            H.check(lib.b200h_group_norm_rows(x.data_ptr(), rows.data_ptr(), w["final.norm"].data_ptr(), n_rows, W, 1, eps, xn.data_ptr(),
+                                              dt, st), "group_norm_rows")
+            return self._logits(xn)
+
+    def gated_linear_mixer(self, i, proj, c, run=None, m=None, p=None):
+        """Gated linear attention of layer i over its columns of a stacked projection, proj [n, q | k | v | g | a1] (T): the per-channel
+        decays from the low-rank columns, the per-head recurrence on the sequence's float state, then the per-head norm and
+        silu(g).  Returns [n, heads * vdim] (T)."""
+        r = i if run is None else run
+        m = self.spec.layers[i].mixer if m is None else m
+        p = f"l{i}." if p is None else p
+        w, lib, dev, n, st = self.w, self.lib, self.device, c.n, self._stream()
+        HD, HV = m.heads * m.dim, m.heads * m.vdim
+        ld, es, base = proj.stride(0), proj.element_size(), proj.data_ptr()
+        decay = torch.empty(n, HD, dtype=torch.float32, device=dev)
+        with self.timed("low-rank decay"):
+            H.check(lib.b200h_low_rank_decay(base + es * 2 * (HD + HV), ld, w[p + "a2"].data_ptr(), w[p + "a2.b"].data_ptr(), n, HD, m.rank, m.tau,
+                                             decay.data_ptr(), self.dt, st), "low_rank_decay")
+        o = torch.empty(n, HV, dtype=torch.float32, device=dev)
+        with self.timed("gated linear recurrence"):
+            H.check(lib.b200h_gated_linear_scan(base, base + es * HD, base + es * 2 * HD, ld, m.dim ** -0.5, decay.data_ptr(),
+                                                c.state.ptr(self.mix_off[r]), c.state.storage.stride(0), c.cu_q.data_ptr(), c.seq_slot.data_ptr(),
+                                                c.batch, m.heads, m.dim, m.vdim, o.data_ptr(), self.dt, st), "gated_linear_scan")
+        y = torch.empty(n, HV, dtype=self.T, device=dev)
+        with self.timed("head norm + gate"):
+            H.check(lib.b200h_group_norm_gate(o.data_ptr(), w[p + "norm"].data_ptr(), base + es * (2 * HD + HV), ld, n, HV, m.heads,
+                                              H.GATE_ACT["silu"], self.spec.norm_eps, y.data_ptr(), self.dt, st), "group_norm_gate")
+        return y
+
+    def rglru_mixer(self, i, h, c, run=None):
+        """RG-LRU of layer i over its input h [n, width] (T): one stacked projection (y | x), the short convolution of x, one batched
+        product over the diagonal blocks for both gates (float result), then the recurrence on the sequence's float state times
+        gelu(y); the scan also advances the convolution's state.  Returns [n, mixer width] (T)."""
+        r = i if run is None else run
+        m, w, lib, dev, T, n = self.spec.layers[i].mixer, self.w, self.lib, self.device, self.T, c.n
+        p, R = f"l{i}.", m.width
+        with self.timed("gemm in"):
+            proj = self._linear(h, w[p + "in"])
+        a = H.RgLruArgs()
+        a.n, a.batch, a.width, a.blocks, a.taps, a.rate = n, c.batch, R, m.blocks, m.conv_taps, m.rate
+        a.y, a.x, a.ld = proj.data_ptr(), proj.data_ptr() + proj.element_size() * R, proj.stride(0)
+        for field, key in (("x_bias", "x.b"), ("y_bias", "y.b"), ("conv", "conv"), ("conv_bias", "conv.b"), ("r_bias", "ra.b"), ("i_bias", "ri.b"),
+                           ("lam", "lam")):
+            setattr(a, field, w[p + key].data_ptr())
+        u, out = torch.empty(n, R, dtype=T, device=dev), torch.empty(n, R, dtype=T, device=dev)
+        a.u, a.out = u.data_ptr(), out.data_ptr()
+        a.conv_state, a.state, a.slot_stride = c.state.ptr(self.conv_off[r]), c.state.ptr(self.mix_off[r]), c.state.storage.stride(0)
+        a.tok_seq, a.cu_q, a.seq_slot = c.tok_seq.data_ptr(), c.cu_q.data_ptr(), c.seq_slot.data_ptr()
+        a.dtype, a.stream = self.dt, self._stream()
+        with self.timed("gated conv"):
+            H.check(lib.b200h_gated_conv(C.byref(a)), "gated_conv")
+        with self.timed("gemm gates"):
+            z = self._bmm(u.view(n, m.blocks, R // m.blocks).transpose(0, 1), w[p + "gates"].transpose(1, 2))
+        a.z = z.data_ptr()
+        with self.timed("real-gated recurrence"):
+            H.check(lib.b200h_real_gated_scan(C.byref(a)), "real_gated_scan")
+        return out
+
     def channel_decay_mixer(self, i, blends, c, run=None, m=None, p=None):
         """Channel-decay recurrence of layer i over the five blends [5, n, width] (T; for r, k, v, the gate and the decay): one batched
         product for r | k | v | g, the decay's two small products around a tanh, the per-channel decays and the per-head recurrence on
@@ -770,6 +967,8 @@ class HybridModel:
             return self.conv_attention_mixer(i, h, c, run=r)
         if kind == "mamba2":
             return self.ssm_mixer(i, h, c, run=r)
+        if kind == "rglru":
+            return self.rglru_mixer(i, h, c, run=r)
         return self.decay_mixer(i, h, c, run=r)
 
     def window_splits(self, n, window, max_pos):
@@ -791,9 +990,9 @@ class HybridModel:
         ld = (keys + 255) // 256 * 256
         return min(ld, (window + 3) // 4 * 4) if window else ld
 
-    def window_mixer(self, i, h, c, run=None, m=None, p=None):
+    def window_mixer(self, i, h, c, run=None, m=None, p=None, proj=None):
         """Windowed attention of layer i (m, p: the spec and weight prefix of one side of a paired mixer): one stacked projection
-        (q | k | v | gate); biases + RMS norm of q and k (over their whole projections, or per head followed by a rotation) + cache
+        (q | k | v | gate; proj: its columns of a wider product that the caller has made already); biases + RMS norm of q and k (over their whole projections, or per head followed by a rotation) + cache
         store in one kernel; then attention over the window or chunk of cached keys with capped scores, distance penalty, the heads'
         scores or softmax weights recombined, a sink, and the output gate.  Returns [n, heads * vdim] (T)."""
         r = i if run is None else run
@@ -801,8 +1000,9 @@ class HybridModel:
         p = f"l{i}." if p is None else p
         w, lib, dev, T, n = self.w, self.lib, self.device, self.T, c.n
         HD, GD, GV, HV = m.heads * m.dim, m.kv_heads * m.dim, m.kv_heads * m.vdim, m.heads * m.vdim
-        with self.timed("gemm in"):
-            proj = self._linear(h, w[p + "in"])
+        if proj is None:
+            with self.timed("gemm in"):
+                proj = self._linear(h, w[p + "in"])
         ld, es, base = proj.stride(0), proj.element_size(), proj.data_ptr()
         f32 = dict(dtype=torch.float32, device=dev)
         a = H.WindowArgs()
@@ -810,6 +1010,8 @@ class HybridModel:
         a.chunk, a.talk_scores, a.gate_heads = m.chunk, int(m.talk_scores), int(m.gate_per_head)
         a.splits = self.window_splits(n, m.span, c.max_pos)
         a.scale, a.softcap, a.eps = m.scale, m.softcap, self.spec.norm_eps
+        if m.q_temp is not None:
+            a.q_temp_coef, a.q_temp_every = m.q_temp
         a.q, a.k, a.v, a.ld = base, base + es * HD, base + es * (HD + GD), ld
         if m.bias:
             a.bias = w[p + "in.b"].data_ptr()
@@ -931,9 +1133,22 @@ class HybridModel:
                                               self.spec.norm_eps, y.data_ptr(), self.dt, st), "gate_group_norm")
         return y
 
+    def gated_mlp(self, h, up, down, name="gated feed-forward"):
+        """down(silu(gate h) * up h) over h [n, width] (T) with gate and up stacked in one matrix -> [n, width] (T)."""
+        with self.timed(f"gemm {name}"):
+            gu = self._linear(h, up)
+        n, ff = h.shape[0], up.shape[0] // 2
+        a = torch.empty(n, ff, dtype=self.T, device=self.device)
+        with self.timed("silu * up"):
+            H.check(self.lib.b200h_silu_mul_rows(gu.data_ptr(), n, ff, a.data_ptr(), self.dt, self._stream()), "silu_mul_rows")
+        with self.timed(f"gemm {name}"):
+            return self._linear(a, down)
+
     def dense_mlp(self, i, h):
         """Dense feed-forward of layer i over its input h [n, width] (T): down(act(up h)) -> [n, width] (T)."""
         f, w = self.spec.layers[i].mlp, self.w
+        if f.act == "silu_gate":
+            return self.gated_mlp(h, w[f"l{i}.up"], w[f"l{i}.down"])
         if f.act not in ("relu2", "xielu"):
             raise NotImplementedError(f"activation {f.act!r}")
         with self.timed("gemm up"):
@@ -1103,8 +1318,8 @@ class HybridModel:
                                                 w[p + "correction"].data_ptr() if f.correction else None, n, W, f.experts, f.top, f.groups,
                                                 f.keep, f.group_top, int(f.renorm), f.scale, ids.data_ptr(), wts.data_ptr(), st), "route_grouped")
             else:
-                H.check(lib.b200h_route_scored(src.data_ptr(), src_dt, w[p + "router"].data_ptr(), n, W, f.experts, f.top, H.SCORE_FN[f.score],
-                                               ids.data_ptr(), wts.data_ptr(), st), "route")
+                H.check(lib.b200h_route_scored(src.data_ptr(), src_dt, w[p + "router"].data_ptr(), w[p + "router.b"].data_ptr() if f.router_bias else None,
+                                               n, W, f.experts, f.top, H.SCORE_FN[f.score], ids.data_ptr(), wts.data_ptr(), st), "route")
         out = torch.empty(n, f.top, W, dtype=torch.float32, device=dev)
         self.last_routing = (ids, wts)
         capturing = dev.type == "cuda" and torch.cuda.is_current_stream_capturing()      # the grouped path reads counts on the host

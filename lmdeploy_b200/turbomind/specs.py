@@ -178,6 +178,8 @@ class WindowAttentionSpec:
     talk_scores: bool = False
     sink: bool = False
     gate_per_head: bool = False
+    # (coef, every): a query at position p is multiplied by 1 + coef * ln(1 + floor((p + 1) / every))
+    q_temp: tuple = None
     kind = "window_attention"
 
     @property
@@ -252,11 +254,36 @@ class ChannelDecaySpec:
 
 
 @dataclass(frozen=True)
+class GatedLinearSpec:
+    """Gated linear attention: per head S <- diag(alpha_t) S + k_t v_t^T, o_t = S^T q_t / sqrt(dim) (read after the update) with S a
+    [dim, vdim] float matrix and a decay per key channel alpha = sigmoid(A2 (A1 h) + b)^(1 / tau) of inner size `rank`; every head's o
+    is RMS-normed over vdim with a weight all heads share, times silu(W_g h), then projected."""
+    heads: int
+    dim: int
+    vdim: int
+    rank: int
+    tau: float
+    kind = "gated_linear"
+
+
+@dataclass(frozen=True)
+class RgLruSpec:
+    """Griffin's recurrent block: branches y = gelu_tanh(W_y h + b) and u = causal convolution (taps per channel, bias, no activation)
+    of W_x h + b, both of `width` channels; r and i are sigmoids of block-diagonal maps of u (`blocks` square blocks);
+    log a = -rate * r * softplus(lam), S <- a S + sqrt(1 - a^2) * i * u (float, one number per channel); S * y is projected."""
+    width: int
+    blocks: int
+    conv_taps: int
+    rate: float = 8.0
+    kind = "rglru"
+
+
+@dataclass(frozen=True)
 class PairedMixerSpec:
     """Two mixers side by side on the same input, each with an output projection of its own; the result is
     (rms(left) * w_left + rms(right) * w_right) / 2 with RMS norms over the model width."""
     left: object                        # WindowAttentionSpec
-    right: object                       # ChannelDecaySpec
+    right: object                       # ChannelDecaySpec (shared-norm blocks) | GatedLinearSpec (sandwich blocks)
     kind = "paired"
 
 
@@ -265,7 +292,8 @@ class RoutedExpertsSpec:
     experts: int
     top: int
     ff: int
-    score: str = "softmax"        # router scores: 'softmax' over all experts | 'sigmoid' of every logit on its own
+    score: str = "softmax"        # router scores: 'softmax' over all experts | 'sigmoid' of every logit on its own |
+    #                               'softmax_chosen': softmax over the chosen logits only
     act: str = "silu_gate"        # expert: 'silu_gate' = down(silu(gate h) * up h) | 'relu2' = down(relu(up h)^2), no gate matrix
     scale_input: bool = False     # the router's score multiplies the expert's input instead of its output
     # a router that chooses among groups (score 'sigmoid' only): a learned correction joins the scores for the CHOICE; the experts form
@@ -278,13 +306,16 @@ class RoutedExpertsSpec:
     group_top: int = 2
     renorm: bool = False
     scale: float = 1.0
+    router_bias: bool = False     # a learned bias on the router's logits
+    shared: int = 0               # > 0: an expert of this inner size (same activation) runs for every token and is added
     kind = "moe"
 
 
 @dataclass(frozen=True)
 class DenseMlpSpec:
     """down(act(up h)); act 'relu2' = the square of relu; 'xielu' = softplus(p) z^2 + z / 2 for z > 0 and
-    (1/2 + softplus(q)) (exp(z) - 1 - z) + z / 2 otherwise, with the two learned numbers p, q of the layer's 'mlp.act'."""
+    (1/2 + softplus(q)) (exp(z) - 1 - z) + z / 2 otherwise, with the two learned numbers p, q of the layer's 'mlp.act';
+    'silu_gate' = down(silu(gate h) * up h) with a gate matrix beside up."""
     ff: int
     act: str = "relu2"
     kind = "dense"
@@ -301,7 +332,7 @@ class HashedBigramSpec:
 
 @dataclass(frozen=True)
 class HybridLayerSpec:
-    mixer: object                       # Latent / Decay / Window / Conv attention spec | SsmSpec | PairedMixerSpec
+    mixer: object                       # Latent / Decay / Window / Conv attention spec | SsmSpec | PairedMixerSpec | RgLruSpec
     mlp: object = None                  # RoutedExpertsSpec | DenseMlpSpec | None: the layer has no feed-forward
 
 
@@ -335,6 +366,8 @@ class HybridSpec:
     #              previous token's normed row (h + (h' - h) * shift, a learned vector per layer), the feed-forward the row itself.
     plain_norms: bool = False           # norm weights are stored as the full factor also in pre-norm / parallel / shared-norm blocks
     bigram: HashedBigramSpec = None     # the embedding adds a hashed row of a second table chosen by the previous token
+    # 'sandwich' blocks: a norm before AND after each sublayer (plain weights), x <- x + n1b(mixer(n1(x))), x <- x + n2b(ff(n2(x))).
+    logit_scale: float = 1.0
     hybrid = True
 
     @property
@@ -506,5 +539,64 @@ def fogizen_spec(cfg, name="fogizen", tensor_shapes=None):
                       session_len=int(cfg.get("session_len", 0)), block="shared_norm", plain_norms=True, bigram=bigram)
 
 
+def _duparax_left(m):
+    heads, kv_heads = int(m["heads"]), int(m["kv_heads"])
+    if heads % kv_heads:
+        raise ValueError(f"{heads} query heads do not divide into {kv_heads} key/value heads")
+    t = m.get("q_temp")
+    if t is not None and not float(t["every"]) > 0:
+        raise ValueError(f"q_temp.every {t['every']}")
+    return WindowAttentionSpec(heads, kv_heads, int(m["dim"]), int(m["vdim"]), float(m["scale"]), qk_norm=False, bias=True, distance_bias=False,
+                               talking_heads=False, gate=False, q_temp=(float(t["coef"]), float(t["every"])) if t is not None else None)
+
+
+def _duparax_mixer(kind, m, rank):
+    """rank: () -> the inner size of the decay's two matrices, asked for only where the mixer has them."""
+    if kind == "parallel":
+        r = m["right"]
+        return PairedMixerSpec(_duparax_left(m["left"]), GatedLinearSpec(int(r["heads"]), int(r["dim"]), int(r["vdim"]), rank(), float(r["tau"])))
+    if kind == "rglru":
+        s = RgLruSpec(int(m["width"]), int(m["blocks"]), int(m["conv"]))
+        if s.width % s.blocks:
+            raise ValueError(f"{s.width} channels in {s.blocks} blocks")
+        return s
+    raise NotImplementedError(f"mixer type {kind!r}")
+
+
+def duparax_spec(cfg, name="duparax", tensor_shapes=None):
+    """config.json of a Duparax checkpoint -> HybridSpec.  Every size and constant is read from the config; the inner size of the
+    decay's two matrices is a tensor's shape ('l<i>.mix.right.a1': [rank, width])."""
+    layers = []
+    for i, entry in enumerate(cfg["layers"]):
+
+        def rank():
+            r = entry["mixer"]["right"]
+            if "rank" in r:
+                return int(r["rank"])
+            if not tensor_shapes:
+                raise ValueError(f"layer {i}: the decay's inner size is neither in the config nor a known tensor shape")
+            return int(tensor_shapes[f"l{i}.mix.right.a1"][0])
+
+        mixer = _duparax_mixer(entry["type"], entry["mixer"], rank)
+        mlp = entry.get("mlp")
+        if mlp is not None:
+            if mlp["kind"] == "dense":
+                mlp = DenseMlpSpec(int(mlp["ff"]), act="silu_gate")
+            elif mlp["kind"] == "moe":
+                r, shared = mlp["router"], mlp.get("shared")
+                mlp = RoutedExpertsSpec(int(r["experts"]), int(r["top"]), int(mlp["expert"]["ff"]), score="softmax_chosen", router_bias=True,
+                                        shared=int(shared["ff"]) if shared else 0)
+                if not 1 <= mlp.top <= mlp.experts:
+                    raise ValueError(f"layer {i}: top {mlp.top} of {mlp.experts} experts")
+            else:
+                raise NotImplementedError(f"feed-forward kind {mlp['kind']!r}")
+        layers.append(HybridLayerSpec(mixer, mlp))
+    return HybridSpec(name=name, arch="duparax", width=int(cfg["width"]), vocab=int(cfg["vocab"]), layers=tuple(layers),
+                      norm_eps=float(cfg["norm"]["eps"]), norm_groups=1, conv_taps=1, embedding_scale=1.0,
+                      session_len=int(cfg.get("session_len", 0)), block="sandwich", plain_norms=True,
+                      logit_scale=float(cfg.get("logit_scale", 1.0)))
+
+
 # config.json "architecture" -> spec builder, for checkpoints that are not HF `architectures` configs
-HYBRID_ARCHITECTURES = {"Gulozen": gulozen_spec, "Bodopel": bodopel_spec, "Lifuzen": lifuzen_spec, "Fogizen": fogizen_spec}
+HYBRID_ARCHITECTURES = {"Gulozen": gulozen_spec, "Bodopel": bodopel_spec, "Lifuzen": lifuzen_spec, "Fogizen": fogizen_spec,
+                        "Duparax": duparax_spec}

@@ -178,15 +178,22 @@ class EmulatedHybridLib:
         return 0
 
     def b200h_route(self, x, router, n, width, experts, top, ids, wts, stream):
-        return self.b200h_route_scored(x, F32, router, n, width, experts, top, 0, ids, wts, stream)
+        return self.b200h_route_scored(x, F32, router, None, n, width, experts, top, 0, ids, wts, stream)
 
-    def b200h_route_scored(self, x, x_dtype, router, n, width, experts, top, score_fn, ids, wts, stream):
+    def b200h_route_scored(self, x, x_dtype, router, bias, n, width, experts, top, score_fn, ids, wts, stream):
         assert x_dtype == F32
         z = _f(x, n, width) @ _f(router, experts, width).T
-        if score_fn == 1:
-            order = np.argsort(-z, -1, kind="stable")[:, :top]          # chosen on the logits: the sigmoid keeps their order
+        if bias:
+            z = z + _f(bias, experts)
+        if score_fn:
+            order = np.argsort(-z, -1, kind="stable")[:, :top]          # chosen on the logits: both score functions keep their order
             _i(ids, n * top).reshape(n, top)[:] = order
-            _f(wts, n, top)[:] = _sigmoid(np.take_along_axis(z, order, -1))
+            chosen = np.take_along_axis(z, order, -1)
+            if score_fn == 2:
+                chosen = np.exp(chosen - chosen.max(-1, keepdims=True))
+                _f(wts, n, top)[:] = chosen / chosen.sum(-1, keepdims=True)
+            else:
+                _f(wts, n, top)[:] = _sigmoid(chosen)
             return 0
         else:
             e = np.exp(z - z.max(-1, keepdims=True))
@@ -260,6 +267,13 @@ class EmulatedHybridLib:
         G, D, V = a.kv_heads, a.dim, a.vdim
         return _f(base + 4 * at * G * D, G, D), _f(base + a.v_off + 4 * at * G * V, G, V)
 
+    @staticmethod
+    def _growth(a, pos):
+        """[n] factors on the queries at positions pos."""
+        if a.q_temp_every == 0:
+            return np.ones(len(pos), np.float32)
+        return (1.0 + a.q_temp_coef * np.log(np.floor((pos + 1) / a.q_temp_every) + 1.0)).astype(np.float32)
+
     def b200h_window_prep(self, args):
         a = args._obj
         assert a.dtype == F32
@@ -271,6 +285,7 @@ class EmulatedHybridLib:
         _f(a.qn, a.n, H * D)[:] = _unit(q, a.eps) * _f(a.q_norm, H * D) if a.q_norm else q
         kn = _unit(k, a.eps) * _f(a.k_norm, G * D) if a.k_norm else k
         seqs, poss = _i(a.tok_seq, a.n), _i(a.tok_pos, a.n)
+        _f(a.qn, a.n, H * D)[:] *= self._growth(a, poss)[:, None]
         for t in range(a.n):
             kd, vd = self._kv(a, int(seqs[t]), int(poss[t]))
             kd[:] = kn[t].reshape(G, D)
@@ -342,7 +357,7 @@ class EmulatedHybridLib:
         seqs, poss = _i(a.tok_seq, a.n), _i(a.tok_pos, a.n)
         qn = _f(a.qn, a.n, H, D)
         for t in range(a.n):
-            qn[t] = self._rot(q[t], int(poss[t]), holder)
+            qn[t] = self._rot(q[t], int(poss[t]), holder) * self._growth(a, poss[t:t + 1])
             kd, vd = self._kv(a, int(seqs[t]), int(poss[t]))
             kd[:] = self._rot(k[t], int(poss[t]), holder)
             vd[:] = v[t].reshape(G, V)
@@ -462,6 +477,88 @@ class EmulatedHybridLib:
             chosen = chosen / (chosen.sum(-1, keepdims=True) + np.float32(1e-20))
         _i(ids, n * top).reshape(n, top)[:] = order
         _f(wts, n, top)[:] = chosen * np.float32(scale)
+        return 0
+
+    # ---- blocks with a norm on both ends of a sublayer, gated linear attention, real-gated diagonal recurrence
+    def b200h_normed_residual_norm(self, x, left, right, wl, wr, branch_scale, m, ff, parts, w_post, w_next, n, width, eps, h, hf, dtype, stream):
+        assert dtype == F32
+        X = _f(x, n, width)
+        if left or m or ff:
+            y = np.zeros((n, width), np.float32)
+            if left:
+                y += np.float32(branch_scale) * (_unit(_f(left, n, width), eps) * _f(wl, width) + _unit(_f(right, n, width), eps) * _f(wr, width))
+            if m:
+                y += _f(m, n, width)
+            if ff:
+                y += _f(ff, n, parts, width).sum(1)
+            X += _unit(y, eps) * _f(w_post, width)
+        for out in (h, hf):
+            if out:
+                _f(out, n, width)[:] = _unit(X, eps) * _f(w_next, width)
+        return 0
+
+    def b200h_low_rank_decay(self, low, ld, a, bias, n, channels, rank, tau, decay, dtype, stream):
+        z = _rows(low, n, ld, rank) @ _f(a, rank, channels) + _f(bias, channels)
+        _f(decay, n, channels)[:] = np.exp(-np.logaddexp(0, -z) / np.float32(tau))
+        return 0
+
+    def b200h_gated_linear_scan(self, q, k, v, ld, q_scale, decay, state, slot_stride, cu_q, seq_slot, batch, heads, dim, vdim, out, dtype, stream):
+        cu, slots = _i(cu_q, batch + 1), _i(seq_slot, batch)
+        n = int(cu[batch])
+        Q, K, Vv = _rows(q, n, ld, heads * dim), _rows(k, n, ld, heads * dim), _rows(v, n, ld, heads * vdim)
+        Wd, O = _f(decay, n, heads * dim), _f(out, n, heads, vdim)
+        for s in range(batch):
+            S = _f(int(state) + 4 * int(slots[s]) * slot_stride, heads, vdim, dim)            # [head][value][key]
+            for t in range(cu[s], cu[s + 1]):
+                for hh in range(heads):
+                    ks, vs = slice(hh * dim, (hh + 1) * dim), slice(hh * vdim, (hh + 1) * vdim)
+                    S[hh] = S[hh] * Wd[t, ks] + np.outer(Vv[t, vs], K[t, ks])
+                    O[t, hh] = S[hh] @ (Q[t, ks] * np.float32(q_scale))
+        return 0
+
+    def b200h_gated_conv(self, args):
+        a = args._obj
+        assert a.dtype == F32
+        X = _rows(a.x, a.n, a.ld, a.width) + (_f(a.x_bias, a.width) if a.x_bias else np.float32(0))
+        cu, slots = _i(a.cu_q, a.batch + 1), _i(a.seq_slot, a.batch)
+        kept = {}                           # the state is advanced by the scan: put back what _conv_rows advances
+        for s in range(a.batch):
+            st = _f(int(a.conv_state) + 4 * int(slots[s]) * a.slot_stride, a.taps - 1, a.width)
+            kept[s] = (st, st.copy())
+        _f(a.u, a.n, a.width)[:] = self._conv_rows(X, _f(a.conv, a.width, a.taps), _f(a.conv_bias, a.width) if a.conv_bias else None, a.conv_state,
+                                                   a.slot_stride, cu, slots, a.batch, a.taps)
+        for st, old in kept.values():
+            st[:] = old
+        return 0
+
+    def b200h_real_gated_scan(self, args):
+        a = args._obj
+        n, R, size = a.n, a.width, a.width // a.blocks
+        Z = _f(a.z, a.blocks, n, 2, size).transpose(2, 1, 0, 3).reshape(2, n, R)
+        bias = lambda p: _f(p, R) if p else np.float32(0)
+        r, gate = _sigmoid(Z[0] + bias(a.r_bias)), _sigmoid(Z[1] + bias(a.i_bias))
+        la = (-np.float32(a.rate) * np.logaddexp(0, _f(a.lam, R)) * r).astype(np.float32)
+        U, X = _f(a.u, n, R), _rows(a.x, n, a.ld, R) + bias(a.x_bias)
+        y = _rows(a.y, n, a.ld, R) + bias(a.y_bias)
+        y = 0.5 * y * (1 + np.tanh(np.sqrt(2 / np.pi) * (y + 0.044715 * y ** 3)))
+        O = _f(a.out, n, R)
+        cu, slots = _i(a.cu_q, a.batch + 1), _i(a.seq_slot, a.batch)
+        for s in range(a.batch):
+            lo, hi = cu[s], cu[s + 1]
+            if lo == hi:
+                continue
+            S = _f(int(a.state) + 4 * int(slots[s]) * a.slot_stride, R)
+            for t in range(lo, hi):
+                S[:] = np.exp(la[t]) * S + np.sqrt(-np.expm1(2 * la[t])) * gate[t] * U[t]
+                O[t] = S * y[t]
+            st = _f(int(a.conv_state) + 4 * int(slots[s]) * a.slot_stride, a.taps - 1, R)
+            full = np.concatenate([st, X[lo:hi]], 0)
+            st[:] = full[full.shape[0] - (a.taps - 1):]
+        return 0
+
+    def b200h_silu_mul_rows(self, gu, n, cols, out, dtype, stream):
+        G = _f(gu, n, 2, cols)
+        _f(out, n, cols)[:] = G[:, 0] * _sigmoid(G[:, 0]) * G[:, 1]
         return 0
 
     # ---- parallel blocks, convolved rotary attention, state-space mixer
