@@ -112,6 +112,23 @@ def fogizen_bench_config(z, chunk=2048):
                        for i in range(len(HYBRID_LAYERS))]}
 
 
+def duparax_bench_config(z):
+    """A Duparax config.json (dict) of size `z`: the layer pattern of the Gulozen bench, with a paired mixer (the dense decoder's head
+    geometry on its attention side, width / 64 heads of 64 x 64 gated linear attention with decay matrices of inner size 64 on the
+    other) where that has attention, and an RG-LRU of the model's width in 16 blocks with 4 taps where it has the recurrent layer; the
+    first layer's feed-forward is dense with the active size of the routed ones (top * ff), the others have eight gated experts of
+    which two are chosen beside a shared expert of the same size."""
+    d = z["dense"]
+    left = {"heads": d["heads"], "kv_heads": d["kv_heads"], "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "q_temp": {"coef": 0.1, "every": 1024}}
+    right = {"heads": z["width"] // 64, "dim": 64, "vdim": 64, "rank": 64, "tau": 16.0}
+    lru = {"width": z["width"], "blocks": 16, "conv": 4}
+    moe = {"kind": "moe", "expert": {"ff": z["ff"]}, "router": {"experts": z["experts"], "top": z["top"]}, "shared": {"ff": z["ff"]}}
+    dense = {"kind": "dense", "ff": z["top"] * z["ff"]}
+    return {"architecture": "Duparax", "norm": {"eps": 1e-6}, "vocab": HYBRID_VOCAB, "width": z["width"], "logit_scale": 0.5,
+            "layers": [{"type": "rglru" if t == "lightning" else "parallel", "mixer": lru if t == "lightning" else {"left": left, "right": right},
+                        "mlp": dense if i == 0 else moe} for i, t in enumerate(HYBRID_LAYERS)]}
+
+
 def _hybrid_leg(torch, spec, batch, ctx, steps, warm, session, blocks):
     """One hybrid decoder through its engine: throughput, then per-operator device time (eight more decode steps, then one fresh
     4096-row prefill step, bracketed by CUDA events)."""
@@ -119,7 +136,8 @@ def _hybrid_leg(torch, spec, batch, ctx, steps, warm, session, blocks):
     from lmdeploy_b200.turbomind.engine import TurboMind
     eng = TurboMind(spec, TurbomindEngineConfig(dtype="bfloat16", max_batch_size=batch, session_len=session, cache_max_entry_count=blocks,
                                                 max_prefill_token_num=8192), seed=0)
-    _engine_prefill_once(torch, eng, HYBRID_VOCAB, 4, 1024)      # untimed: the library's kernels and the vendor GEMMs load on first use
+    # untimed: the library's kernels and the vendor GEMMs load on first use, and the allocator sees a step of the timed size
+    _engine_prefill_once(torch, eng, HYBRID_VOCAB, batch, ctx)
     res, seqs = _engine_throughput(torch, eng, HYBRID_VOCAB, batch, ctx, steps, warm)
     res["weight_bytes"] = eng.model.weight_bytes
     eng.model.events = []
@@ -177,7 +195,7 @@ def run_hybrid(args):
     from lmdeploy_b200.messages import TurbomindEngineConfig
     from lmdeploy_b200.turbomind import ModelSpec
     from lmdeploy_b200.turbomind.engine import TurboMind
-    from lmdeploy_b200.turbomind.specs import bodopel_spec, fogizen_spec, gulozen_spec, lifuzen_spec
+    from lmdeploy_b200.turbomind.specs import bodopel_spec, duparax_spec, fogizen_spec, gulozen_spec, lifuzen_spec
     z = HYBRID_SIZES[args.hybrid]
     batch, ctx, steps, warm = args.hybrid_batch, args.hybrid_ctx, args.steps, max(args.warmup, 3)
     session = 2 * ctx + warm + steps + 16
@@ -192,6 +210,8 @@ def run_hybrid(args):
             spec = lifuzen_spec(lifuzen_bench_config(z), name=f"lifuzen-{args.hybrid}")
         elif args.hybrid_design == "fogizen":
             spec = fogizen_spec(fogizen_bench_config(z), name=f"fogizen-{args.hybrid}")
+        elif args.hybrid_design == "duparax":
+            spec = duparax_spec(duparax_bench_config(z), name=f"duparax-{args.hybrid}")
         else:
             spec = gulozen_spec(hybrid_config(z), name=f"gulozen-{args.hybrid}")
         out["hybrid"] = _hybrid_leg(torch, spec, batch, ctx, steps, warm, session, blocks)
@@ -203,6 +223,10 @@ def run_hybrid(args):
             # the closest existing model -- parallel blocks, two-pass attention with a sink, a scanned recurrence, sigmoid-routed experts
             out["closest"] = dict(_hybrid_leg(torch, lifuzen_spec(lifuzen_bench_config(z), name=f"lifuzen-{args.hybrid}"), batch, ctx, steps,
                                               warm, session, blocks), design="lifuzen")
+        if args.hybrid_design == "duparax":
+            # the closest existing model -- paired mixers of attention and a channel-decay recurrence, dense and routed gated feed-forwards
+            out["closest"] = dict(_hybrid_leg(torch, fogizen_spec(fogizen_bench_config(z), name=f"fogizen-{args.hybrid}"), batch, ctx, steps,
+                                              warm, session, blocks), design="fogizen")
         d = z["dense"]
         dspec = ModelSpec(f"dense-{args.hybrid}", "llama", d["hidden"], len(HYBRID_LAYERS), d["heads"], d["kv_heads"], d["inter"], HYBRID_VOCAB,
                           1e4, weight_format="fp16")
@@ -237,12 +261,14 @@ def parse():
     ap.add_argument("--hybrid", default=None, choices=list(HYBRID_SIZES),
                     help="instead of the default workload: prefill and decode tokens/s of a hybrid decoder of this size (--hybrid-design) "
                          "beside the dense decoder of equal size, both through the engine (random weights)")
-    ap.add_argument("--hybrid-design", default="gulozen", choices=["gulozen", "bodopel", "lifuzen", "fogizen"],
+    ap.add_argument("--hybrid-design", default="gulozen", choices=["gulozen", "bodopel", "lifuzen", "fogizen", "duparax"],
                     help="which hybrid design --hybrid builds: Gulozen (latent / decayed linear attention, routed experts), Bodopel "
                          "(windowed attention with grouped key/value heads, dense feed-forward) or Lifuzen (parallel blocks: convolved rotary "
                          "attention with a sink / state-space mixer, sigmoid-routed squared-relu experts; also runs Gulozen of equal size, the "
                          "closest existing model, beside it) or Fogizen (shared-norm blocks with token shift: chunked rotary attention beside a "
-                         "channel-decay recurrence in every layer, dense and group-routed experts; also runs Lifuzen of equal size beside it)")
+                         "channel-decay recurrence in every layer, dense and group-routed experts; also runs Lifuzen of equal size beside it) or Duparax (norms on both ends of "
+                         "every sublayer: attention beside gated linear attention / RG-LRU, dense and routed feed-forwards with a shared expert; "
+                         "also runs Fogizen of equal size beside it)")
     ap.add_argument("--hybrid-batch", type=int, default=32)
     ap.add_argument("--hybrid-ctx", type=int, default=1024)
     ap.add_argument("--no-graph", action="store_true", help="do not capture the step in a CUDA graph")

@@ -6,52 +6,6 @@
 // Number formats: projections (T) are read once; decays, gates, the recurrence and its state are float.  The convolution's output u
 // is T: it is the operand of the gates' block-diagonal product, and the recurrence reads the same rounded values.
 
-// decay[t, c] = sigmoid(sum_k a[k, c] low[t, k] + bias[c])^(1 / tau) = exp(-softplus(-z) / tau).  A block takes ROWS rows and
-// blockDim.x channels; the rows' low-rank vectors sit in shared memory as [rank][ROWS], a thread reads its column of `a` once for all.
-template <typename T, int ROWS>
-__global__ void __launch_bounds__(256) low_rank_decay_kernel(const T* __restrict__ low, int64_t ld, const T* __restrict__ a,
-                                                            const float* __restrict__ bias, int n, int channels, int rank, float inv_tau,
-                                                            float* __restrict__ decay)
-{
-    extern __shared__ __align__(16) float lrd_smem[];
-    const int t0 = blockIdx.y * ROWS, c = blockIdx.x * blockDim.x + threadIdx.x;
-    for (int i = threadIdx.x; i < rank * ROWS; i += blockDim.x) {
-        const int r = i / rank, k = i - r * rank;
-        lrd_smem[k * ROWS + r] = t0 + r < n ? to_f(low[(size_t)(t0 + r) * ld + k]) : 0.f;
-    }
-    __syncthreads();
-    if (c >= channels) return;
-    float z[ROWS];
-    const float b = bias[c];
-#pragma unroll
-    for (int r = 0; r < ROWS; ++r) z[r] = b;
-#pragma unroll 8
-    for (int k = 0; k < rank; ++k) {
-        const float w = to_f(a[(size_t)k * channels + c]);
-        if (ROWS % 4 == 0) {
-#pragma unroll
-            for (int r = 0; r < ROWS; r += 4) {
-                const float4 v = *reinterpret_cast<const float4*>(lrd_smem + k * ROWS + r);
-                z[r] = fmaf(w, v.x, z[r]);
-                z[(r + 1) % ROWS] = fmaf(w, v.y, z[(r + 1) % ROWS]);
-                z[(r + 2) % ROWS] = fmaf(w, v.z, z[(r + 2) % ROWS]);
-                z[(r + 3) % ROWS] = fmaf(w, v.w, z[(r + 3) % ROWS]);
-            }
-        } else {
-#pragma unroll
-            for (int r = 0; r < ROWS; ++r) z[r] = fmaf(w, lrd_smem[k * ROWS + r], z[r]);
-        }
-    }
-#pragma unroll
-    for (int r = 0; r < ROWS; ++r)
-        if (t0 + r < n) decay[(size_t)(t0 + r) * channels + c] = expf(-softplus32(-z[r]) * inv_tau);
-}
-
-__device__ __forceinline__ float gelu_tanh_f(float z)
-{
-    return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * fmaf(0.044715f * z * z, z, z)));       // sqrt(2 / pi)
-}
-
 // V consecutive values of T as float / back
 template <int V> __device__ __forceinline__ void load_vals(const float* p, float (&o)[V])
 {
@@ -72,6 +26,66 @@ template <int V> __device__ __forceinline__ void store_vals(float* p, const floa
 template <int V> __device__ __forceinline__ void store_vals(bf16* p, const float (&v)[V])
 {
     if (V == 2) *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(v[0], v[V - 1]); else p[0] = from_f<bf16>(v[0]);
+}
+
+// decay[t, c] = sigmoid(sum_k a[k, c] low[t, k] + bias[c])^(1 / tau) = exp(-softplus(-z) / tau).  A block takes ROWS rows and
+// V * blockDim.x channels; the rows' low-rank vectors sit in shared memory as [rank][ROWS], a thread reads its V columns of `a` once
+// for all of them and keeps ROWS * V sums in registers.
+template <typename T, int ROWS, int V>
+__global__ void __launch_bounds__(128) low_rank_decay_kernel(const T* __restrict__ low, int64_t ld, const T* __restrict__ a,
+                                                            const float* __restrict__ bias, int n, int channels, int rank, float inv_tau,
+                                                            float* __restrict__ decay)
+{
+    extern __shared__ __align__(16) float lrd_smem[];
+    constexpr int Q = ROWS % 4 == 0 ? 4 : 1;                  // rows per shared-memory read
+    const int t0 = blockIdx.y * ROWS, c = (blockIdx.x * blockDim.x + threadIdx.x) * V;
+    for (int i = threadIdx.x; i < rank * ROWS; i += blockDim.x) {
+        const int r = i / rank, k = i - r * rank;
+        lrd_smem[k * ROWS + r] = t0 + r < n ? to_f(low[(size_t)(t0 + r) * ld + k]) : 0.f;
+    }
+    __syncthreads();
+    if (c >= channels) return;
+    float z[ROWS][V];
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+        const float b = bias[c + e];
+#pragma unroll
+        for (int r = 0; r < ROWS; ++r) z[r][e] = b;
+    }
+#pragma unroll 8
+    for (int k = 0; k < rank; ++k) {
+        float w[V];
+        load_vals<V>(a + (size_t)k * channels + c, w);
+#pragma unroll
+        for (int r = 0; r < ROWS; r += Q) {
+            float v[Q];
+            if (Q == 4) {
+                const float4 q = *reinterpret_cast<const float4*>(lrd_smem + k * ROWS + r);
+                v[0] = q.x; v[1 % Q] = q.y; v[2 % Q] = q.z; v[3 % Q] = q.w;
+            } else {
+                v[0] = lrd_smem[k * ROWS + r];
+            }
+#pragma unroll
+            for (int q = 0; q < Q; ++q)
+#pragma unroll
+                for (int e = 0; e < V; ++e) z[r + q][e] = fmaf(w[e], v[q], z[r + q][e]);
+        }
+    }
+#pragma unroll
+    for (int r = 0; r < ROWS; ++r) {
+        if (t0 + r < n) {
+            float d[V];
+#pragma unroll
+            for (int e = 0; e < V; ++e) d[e] = expf(-softplus32(-z[r][e]) * inv_tau);
+            store_vals<V>(decay + (size_t)(t0 + r) * channels + c, d);
+        }
+    }
+}
+
+// 0.5 z (1 + tanh(w)) = z sigmoid(2 w), w = sqrt(2 / pi) (z + 0.044715 z^3)
+__device__ __forceinline__ float gelu_tanh_f(float z)
+{
+    return z / (1.0f + expf(-1.5957691216057308f * fmaf(0.044715f * z * z, z, z)));              // 2 sqrt(2 / pi)
 }
 
 // u[t, c] = conv_bias[c] + sum_j w[c, j] * v[t - taps + 1 + j, c] with v = x + x_bias; v before a sequence's rows of this step comes from

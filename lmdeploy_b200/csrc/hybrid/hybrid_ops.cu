@@ -1610,15 +1610,16 @@ B200H_API int b200h_low_rank_decay(const void* low, int64_t ld, const void* a, c
 {
     if (!low || !a || !bias || !decay || n < 0 || channels <= 0 || rank <= 0 || !(tau > 0.f))
         return fail(B200H_ERR_INVALID_ARG, "low_rank_decay: bad arguments");
-    if (rank > 1024) return fail(B200H_ERR_UNSUPPORTED, "low_rank_decay: rank <= 1024");
+    if (rank > 8192) return fail(B200H_ERR_UNSUPPORTED, "low_rank_decay: rank <= 8192");
     if (n == 0) return 0;
     cudaStream_t st = (cudaStream_t)stream;
-    const int cb = (channels + 255) / 256;
-    // eight rows share a read of `a`; one where that would leave SMs without a block
-#define B200H_LRD(ROWS)                                                                                                               \
-    low_rank_decay_kernel<T, ROWS><<<dim3(cb, (n + ROWS - 1) / ROWS), 256, (size_t)rank * ROWS * sizeof(float), st>>>(                 \
+    // sixteen rows share a read of `a`; one where that would leave SMs without a block.  Two channels per thread where they are aligned
+    const int v = channels % 2 == 0 ? 2 : 1, cb = (channels + 128 * v - 1) / (128 * v);
+    const bool many = (int64_t)cb * n >= 16 * 296 && rank <= 512;
+#define B200H_LRD(ROWS, V)                                                                                                            \
+    low_rank_decay_kernel<T, ROWS, V><<<dim3(cb, (n + ROWS - 1) / ROWS), 128, (size_t)rank * ROWS * sizeof(float), st>>>(              \
         (const T*)low, ld, (const T*)a, (const float*)bias, n, channels, rank, 1.0f / tau, (float*)decay)
-    B200H_DISPATCH_T(dtype, if ((int64_t)cb * n >= 4096) B200H_LRD(8); else B200H_LRD(1));
+    B200H_DISPATCH_T(dtype, if (many && v == 2) B200H_LRD(16, 2); else if (many) B200H_LRD(16, 1); else if (v == 2) B200H_LRD(1, 2); else B200H_LRD(1, 1));
 #undef B200H_LRD
     return launched("low_rank_decay");
 }
