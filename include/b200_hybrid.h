@@ -5,7 +5,8 @@
  * and a token shift, two mixers side by side, chunked rotary attention with scores mixed across heads, a recurrence with a
  * decay per key channel and token, a router that chooses among groups of experts; blocks that norm a sublayer's input and its
  * output, queries that grow with their position, gated linear attention, a real-gated diagonal recurrence, a router whose
- * softmax runs over the chosen experts) for sm_100a.
+ * softmax runs over the chosen experts; blocks of parallel residual streams, differential attention, a sliding window that keeps
+ * the first tokens, retention, the gated delta rule) for sm_100a.
  *
  * Conventions shared by all entries: raw device pointers, sizes as int, `stream` a cudaStream_t, return 0 on success, a
  * negative b200h_status for refused arguments, a positive cudaError_t for a failed launch; b200h_last_error() says why.
@@ -30,12 +31,14 @@
 
 enum b200h_status { B200H_ERR_INVALID_ARG = -1, B200H_ERR_UNSUPPORTED = -2 };
 
-/* Rotation of interleaved pairs (2i, 2i+1), i < pairs, by the angle position * freqs[i]; cos and sin times magnitude.
+/* Rotation of interleaved pairs (2i, 2i+1) -- or, halves 1, of pairs (i, i + pairs) --, i < pairs, by the angle position * freqs[i]; cos
+ * and sin times magnitude.  (halves is understood by b200h_head_rope_prep and b200h_retention_prep; the other entries refuse it.)
  * freqs: `pairs` doubles in device memory. */
 typedef struct b200h_rotary {
     const void* freqs;
     int pairs;
     float magnitude;
+    int halves;
 } b200h_rotary;
 
 /* One latent-attention layer of one step.
@@ -173,7 +176,12 @@ B200H_API int b200h_relu2(void* x, int64_t count, int dtype, void* stream);
  *   weight_h <- sum_g talk[h, g] * weight_g if talk;  out_h = sum_j weight_h(j) * v_j;
  *   y = out * sigmoid(gate) if gate.
  * Cache entry of a position inside its page (page address + layer_off): the normed key as T at [pos % block_len][kv_heads * dim],
- * and, v_off bytes further, the value as T at [pos % block_len][kv_heads * vdim]. */
+ * and, v_off bytes further, the value as T at [pos % block_len][kv_heads * vdim].
+ * keep_first > 0 (with a window): every j < keep_first stays visible too, so a row sees at most window + keep_first keys.
+ * maps 2 (differential attention): heads * 2 queries and kv_heads * 2 keys, laid out head by head as [map 1, map 2], over kv_heads values;
+ *   a softmax per map and out_h = sum_j (weight_h1(j) - lambda * weight_h2(j)) * v_j.  Where sizes below say `heads` for queries, scores
+ *   and their statistics (qn, scores, ml, sink) read heads * maps, for keys kv_heads * maps.
+ * out_norm 1: every head's out is divided by sqrt(mean(out^2) + eps) over vdim.  out is multiplied by out_scale. */
 typedef struct b200h_window_args {
     int n, heads, kv_heads, dim, vdim, block_len, window, splits;
     float scale, softcap, eps;
@@ -192,9 +200,9 @@ typedef struct b200h_window_args {
     int64_t ld_gate;
     void* ml;                /* float [n, heads, splits, 2] scratch */
     void* o_part;            /* float [n, splits, heads * vdim] scratch */
-    void* scores;            /* float [n, heads, score_ld] scratch: a row's scores, indexed by key position - the row's first visible key */
-    int64_t score_ld;        /* >= the most keys a row of the step sees: min(window, largest position + 1), all positions when window is 0 */
-    void* y;                 /* T [n, heads * vdim]: out of b200h_window_attention */
+    void* scores;            /* float [n, heads, score_ld] scratch: the score of a row's i-th visible key at index i */
+    int64_t score_ld;        /* >= the most keys a row of the step sees: min(window + keep_first, largest position + 1), all positions when window is 0 */
+    void* y;                 /* T [n, heads * vdim], rows ld_y apart: out of b200h_window_attention */
     const void* tok_seq;     /* int [n] */
     const void* tok_pos;     /* int [n] */
     const void* block_ptrs;  /* int64: page addresses, entry s's pages from cu_blocks[s] */
@@ -208,6 +216,12 @@ typedef struct b200h_window_args {
     int gate_heads;          /* 1: gate is T [n, ld_gate] with ONE column per head instead of one per output column */
     float q_temp_coef;       /* the prep entries multiply a query at position p by 1 + q_temp_coef * ln(1 + floor((p + 1) / q_temp_every)), */
     double q_temp_every;     /* after bias, norm and rotation; q_temp_every 0: by one */
+    int maps;                /* 0 or 1: one softmax per head; 2: two, subtracted */
+    int keep_first;
+    int out_norm;
+    float lambda;            /* maps 2: factor on the second map's weights */
+    float out_scale;         /* factor on the output (1: none) */
+    int64_t ld_y;            /* row stride of y; 0: heads * vdim */
 } b200h_window_args;
 /* Bias, norm of query and key, cache store of key and value (fills qn). */
 B200H_API int b200h_window_prep(const b200h_window_args* args);
@@ -389,5 +403,72 @@ B200H_API int b200h_real_gated_scan(const b200h_rglru_args* args);
 
 /* out[t, i] = silu(gu[t, i]) * gu[t, cols + i] as T [n, cols]; gu T [n, 2 * cols]: between the stacked gate | up product and the down product. */
 B200H_API int b200h_silu_mul_rows(const void* gu, int n, int cols, void* out, int dtype, void* stream);
+
+/* out[t, i] = act(gu[t, i]) * gu[t, cols + i]; act 0: silu (as above), 1: the tanh form of gelu. */
+B200H_API int b200h_gate_mul_rows(const void* gu, int n, int cols, int act, void* out, int dtype, void* stream);
+
+/* ---- blocks of parallel residual streams, retention, gated delta rule ---- */
+
+/* b200h_group_norm_gate with rows of y ld_y apart and w optional (NULL: one). */
+B200H_API int b200h_group_norm_gate_rows(const void* o, const void* w, const void* gate, int64_t ld_gate, int n, int count, int groups, int act,
+                                         float eps, void* y, int64_t ld_y, int dtype, void* stream);
+
+/* e = scale * table[tokens[t]], e <- e / rms(e) * w_embed if w_embed;  x[t, s] = e for every stream s (x float [n, streams, width]);
+ * u = sum_s read[s] e;  h[t] = u / rms(u) * w_next as T.  read float [streams]; norm weights hold the full factor. */
+B200H_API int b200h_embed_streams(const void* tokens, const void* table, float scale, const void* w_embed, void* x, int streams, const void* read,
+                                  const void* w_next, int n, int width, float eps, void* h, int dtype, void* stream);
+
+/* Block b = 0 .. count - 1 takes row t = rows ? rows[b] : b of x (float [.., streams, width], streams <= 8):
+ *   with y (T [.., width]):  x[t, d] <- sum_s mix[s, d] x[t, s] + out[d] * (y[t] * ls), all d from the old streams (ls float [width] or NULL:
+ *   one; mix float [streams, streams], out float [streams]); written back if `write`;
+ *   then u = sum_s read[s] x[t, s] (read NULL: the plain sum) -> u[b] (float, optional) and h[b] = u / rms(u) * w_next (T, optional). */
+B200H_API int b200h_join_streams(void* x, int streams, const void* y, const void* ls, const void* mix, const void* out, const void* read,
+                                 const void* w_next, const void* rows, int count, int width, float eps, int write, void* u, void* h, int dtype,
+                                 void* stream);
+
+/* qk (float [n, 2 * heads * dim]) = rotated q | rotated k * k_scale; q, k: T columns of a projection with row stride ld. */
+B200H_API int b200h_retention_prep(const void* q, const void* k, int64_t ld, int n, int heads, int dim, float k_scale, const b200h_rotary* rot,
+                                   const void* tok_pos, void* qk, int dtype, void* stream);
+
+/* Per head S <- decay[h] S + k v^T, out = S^T q (float [n, heads * vdim]); qk from b200h_retention_prep, v T with row stride ld_v;
+ * decay float [heads]; state float [heads, vdim, dim] at state + seq_slot[s] * slot_stride, read and advanced. */
+B200H_API int b200h_retention_scan(const void* qk, const void* v, int64_t ld_v, const void* decay, void* state, int64_t slot_stride, const void* cu_q,
+                                   const void* seq_slot, int batch, int heads, int dim, int vdim, void* out, int dtype, void* stream);
+
+/* decay[t, h * dim + i] = exp(-rate[h] * softplus(z)), z = sum_k a[k, h * dim + i] * low[t, k] + bias[h * dim + i] (float [n, heads * dim]);
+ * low T [n, rank] with row stride ld, a T [rank, heads * dim], bias float [heads * dim], rate float [heads]. */
+B200H_API int b200h_low_rank_rate_decay(const void* low, int64_t ld, const void* a, const void* bias, const void* rate, int n, int heads, int dim,
+                                        int rank, void* decay, int dtype, void* stream);
+
+/* The gated delta rule of one layer for one step.  channels = 2 * kv_heads * dim + heads * vdim, in the order q | k | v.
+ * b200h_delta_prep:  every channel c of u passes y[t, c] = silu(sum_j conv[j, c] * u[t - taps + 1 + j, c]) (inputs before an entry's first
+ *   row come from conv_state, zeros at a sequence's start);  per key head q <- q_scale * q / sqrt(sum q^2 + unit_eps), k likewise without
+ *   the scale;  qkv = q | k | v, kq = q . k per key head, beta = sigmoid(b).
+ * b200h_delta_scan, head h reading key head h / (heads / kv_heads), S a [dim, vdim] float matrix:
+ *   S <- diag(decay_t) S;  e = beta (v - S^T k);  S <- S + k e^T;  out = S^T q;
+ *   it advances S and then conv_state (the last taps - 1 rows of u, oldest first). */
+typedef struct b200h_delta_args {
+    int n, batch, heads, kv_heads, dim, vdim, taps;
+    float q_scale, unit_eps;
+    const void* u;           /* T: columns q | k | v of a projection, row stride ld */
+    const void* b;           /* T: one column per head, row stride ld */
+    int64_t ld;
+    const void* conv;        /* float [taps, channels] */
+    void* conv_state;        /* float [taps - 1, channels] at conv_state + seq_slot[s] * slot_stride */
+    void* state;             /* float [heads, vdim, dim], same stride */
+    int64_t slot_stride;
+    void* qkv;               /* float [n, channels] */
+    void* kq;                /* float [n, kv_heads] */
+    void* beta;              /* float [n, heads] */
+    const void* decay;       /* float [n, heads * dim] */
+    void* out;               /* float [n, heads * vdim] */
+    const void* tok_seq;     /* int [n] */
+    const void* cu_q;        /* int [batch + 1] */
+    const void* seq_slot;    /* int [batch] */
+    int dtype;
+    void* stream;
+} b200h_delta_args;
+B200H_API int b200h_delta_prep(const b200h_delta_args* args);
+B200H_API int b200h_delta_scan(const b200h_delta_args* args);
 
 #endif

@@ -7,10 +7,11 @@ from ._lib import B200LibraryError
 
 BF16, F32 = 1, 2
 MAX_TAPS = 16
+MAX_STREAMS = 8
 
 
 class Rotary(C.Structure):
-    _fields_ = [("freqs", C.c_void_p), ("pairs", C.c_int), ("magnitude", C.c_float)]
+    _fields_ = [("freqs", C.c_void_p), ("pairs", C.c_int), ("magnitude", C.c_float), ("halves", C.c_int)]
 
 
 class LatentArgs(C.Structure):
@@ -50,7 +51,11 @@ class WindowArgs(C.Structure):
         ("tok_seq", C.c_void_p), ("tok_pos", C.c_void_p), ("block_ptrs", C.c_void_p), ("cu_blocks", C.c_void_p),
         ("layer_off", C.c_int64), ("v_off", C.c_int64), ("dtype", C.c_int), ("stream", C.c_void_p), ("sink", C.c_void_p),
         ("chunk", C.c_int), ("talk_scores", C.c_int), ("gate_heads", C.c_int), ("q_temp_coef", C.c_float), ("q_temp_every", C.c_double),
+        ("maps", C.c_int), ("keep_first", C.c_int), ("out_norm", C.c_int), ("lambda_", C.c_float), ("out_scale", C.c_float), ("ld_y", C.c_int64),
     ]
+
+    def __init__(self, **kw):
+        super().__init__(**dict(dict(out_scale=1.0, maps=1), **kw))
 
 
 class ConvPrepArgs(C.Structure):
@@ -76,8 +81,20 @@ class RgLruArgs(C.Structure):
     ]
 
 
+class DeltaArgs(C.Structure):
+    """b200h_delta_args."""
+    _fields_ = [
+        ("n", C.c_int), ("batch", C.c_int), ("heads", C.c_int), ("kv_heads", C.c_int), ("dim", C.c_int), ("vdim", C.c_int), ("taps", C.c_int),
+        ("q_scale", C.c_float), ("unit_eps", C.c_float), ("u", C.c_void_p), ("b", C.c_void_p), ("ld", C.c_int64), ("conv", C.c_void_p),
+        ("conv_state", C.c_void_p), ("state", C.c_void_p), ("slot_stride", C.c_int64), ("qkv", C.c_void_p), ("kq", C.c_void_p),
+        ("beta", C.c_void_p), ("decay", C.c_void_p), ("out", C.c_void_p), ("tok_seq", C.c_void_p), ("cu_q", C.c_void_p),
+        ("seq_slot", C.c_void_p), ("dtype", C.c_int), ("stream", C.c_void_p),
+    ]
+
+
 SCORE_FN = {"softmax": 0, "sigmoid": 1, "softmax_chosen": 2}
 GATE_ACT = {"sigmoid": 0, "silu": 1}
+MLP_GATE_ACT = {"silu_gate": 0, "gelu_gate": 1}
 EXPERT_ACT = {"silu_gate": 0, "relu2": 1}
 
 _lib = None
@@ -139,6 +156,15 @@ def load():
     lib.b200h_gated_conv.argtypes = [C.POINTER(RgLruArgs)]
     lib.b200h_real_gated_scan.argtypes = [C.POINTER(RgLruArgs)]
     lib.b200h_silu_mul_rows.argtypes = [P, I, I, P, I, P]
+    lib.b200h_gate_mul_rows.argtypes = [P, I, I, I, P, I, P]
+    lib.b200h_group_norm_gate_rows.argtypes = [P, P, P, L64, I, I, I, I, F, P, L64, I, P]
+    lib.b200h_embed_streams.argtypes = [P, P, F, P, P, I, P, P, I, I, F, P, I, P]
+    lib.b200h_join_streams.argtypes = [P, I, P, P, P, P, P, P, P, I, I, F, I, P, P, I, P]
+    lib.b200h_retention_prep.argtypes = [P, P, L64, I, I, I, F, C.POINTER(Rotary), P, P, I, P]
+    lib.b200h_retention_scan.argtypes = [P, P, L64, P, P, L64, P, P, I, I, I, I, P, I, P]
+    lib.b200h_low_rank_rate_decay.argtypes = [P, L64, P, P, P, I, I, I, I, P, I, P]
+    lib.b200h_delta_prep.argtypes = [C.POINTER(DeltaArgs)]
+    lib.b200h_delta_scan.argtypes = [C.POINTER(DeltaArgs)]
     _lib = lib
     return lib
 

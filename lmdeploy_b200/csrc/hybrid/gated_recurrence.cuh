@@ -28,13 +28,14 @@ template <int V> __device__ __forceinline__ void store_vals(bf16* p, const float
     if (V == 2) *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(v[0], v[V - 1]); else p[0] = from_f<bf16>(v[0]);
 }
 
-// decay[t, c] = sigmoid(sum_k a[k, c] low[t, k] + bias[c])^(1 / tau) = exp(-softplus(-z) / tau).  A block takes ROWS rows and
+// z = sum_k a[k, c] low[t, k] + bias[c];  decay[t, c] = sigmoid(z)^(1 / tau) = exp(-softplus(-z) / tau), or, with a rate per head of `dim`
+// channels, exp(-rate[c / dim] softplus(z)).  A block takes ROWS rows and
 // V * blockDim.x channels; the rows' low-rank vectors sit in shared memory as [rank][ROWS], a thread reads its V columns of `a` once
 // for all of them and keeps ROWS * V sums in registers.
 template <typename T, int ROWS, int V>
 __global__ void __launch_bounds__(128) low_rank_decay_kernel(const T* __restrict__ low, int64_t ld, const T* __restrict__ a,
                                                             const float* __restrict__ bias, int n, int channels, int rank, float inv_tau,
-                                                            float* __restrict__ decay)
+                                                            const float* __restrict__ rate, int dim, float* __restrict__ decay)
 {
     extern __shared__ __align__(16) float lrd_smem[];
     constexpr int Q = ROWS % 4 == 0 ? 4 : 1;                  // rows per shared-memory read
@@ -76,7 +77,7 @@ __global__ void __launch_bounds__(128) low_rank_decay_kernel(const T* __restrict
         if (t0 + r < n) {
             float d[V];
 #pragma unroll
-            for (int e = 0; e < V; ++e) d[e] = expf(-softplus32(-z[r][e]) * inv_tau);
+            for (int e = 0; e < V; ++e) d[e] = rate ? expf(-rate[(c + e) / dim] * softplus32(z[r][e])) : expf(-softplus32(-z[r][e]) * inv_tau);
             store_vals<V>(decay + (size_t)(t0 + r) * channels + c, d);
         }
     }

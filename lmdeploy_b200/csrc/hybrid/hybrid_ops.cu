@@ -2,7 +2,8 @@
 // short causal convolution, depth-weighted residual history; window_attention.cuh: pre-norm blocks and windowed attention;
 // ssm.cuh, parallel_block.cuh: the state-space mixer, parallel blocks and convolved rotary attention; token_shift.cuh: shared-norm
 // blocks and the channel-decay recurrence; gated_recurrence.cuh, normed_block.cuh: token-gated recurrences and blocks that norm a
-// sublayer's output) behind a C ABI of their own: libb200hybrid.so.
+// sublayer's output; delta_rule.cuh, stream_block.cuh: retention, the gated delta rule and blocks of parallel residual streams) behind a
+// C ABI of their own: libb200hybrid.so.
 //
 // Number formats.  T is the activation / weight type of the matrix products (float or bf16).  Everything the designs want in
 // 32 bits is float here whatever T is: the residual stream and its history, every norm, rotary angles (double), attention
@@ -16,6 +17,7 @@
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
 #include <stdint.h>
+#include <initializer_list>
 
 namespace b200h {
 
@@ -159,6 +161,7 @@ struct Rotary {
     const double* freqs;      // angle per position of pair i, i < pairs
     int pairs;                // rotated pairs; dimensions from 2 * pairs on pass unchanged
     float magnitude;          // factor on cos and sin
+    int halves;               // 0: pairs (2i, 2i + 1); 1: pairs (i, i + pairs)
 };
 
 __device__ __forceinline__ void rotate_pair(float u, float v, int pos, double f, float mag, float& ru, float& rv)
@@ -798,6 +801,8 @@ __global__ void argmax_kernel(const float* __restrict__ logits, int64_t ld, int 
 #include "token_shift.cuh"
 #include "gated_recurrence.cuh"
 #include "normed_block.cuh"
+#include "delta_rule.cuh"
+#include "stream_block.cuh"
 
 }  // namespace b200h
 
@@ -834,6 +839,7 @@ static Rotary make_rotary(const b200h_rotary* r)
     o.freqs = reinterpret_cast<const double*>(r->freqs);
     o.pairs = r->pairs;
     o.magnitude = r->magnitude;
+    o.halves = r->halves;
     return o;
 }
 
@@ -908,6 +914,7 @@ B200H_API int b200h_latent_prep(const b200h_latent_args* a)
     if (!a || !a->dq || !a->dkv || !a->q_norm || !a->kv_norm || !a->cq || !a->block_ptrs || !a->tok_seq || !a->tok_pos || !a->cu_blocks)
         return fail(B200H_ERR_INVALID_ARG, "latent_prep: bad arguments");
     if (2 * a->rot.pairs > a->rot_dim) return fail(B200H_ERR_INVALID_ARG, "latent_prep: more rotated pairs than rot_dim holds");
+    if (a->rot.halves) return fail(B200H_ERR_UNSUPPORTED, "latent_prep: rotation of interleaved pairs only");
     if (a->n == 0) return 0;
     cudaStream_t st = (cudaStream_t)a->stream;
     B200H_DISPATCH_T(a->dtype, latent_prep_kernel<T><<<a->n, 128, 0, st>>>(
@@ -1153,12 +1160,18 @@ B200H_API int b200h_relu2(void* x, int64_t count, int dtype, void* stream)
     return launched("relu2");
 }
 
+static int window_maps(const b200h_window_args* a) { return a->maps > 1 ? a->maps : 1; }
+
 static int window_args_ok(const b200h_window_args* a, const char** why)
 {
     if (!a || !a->tok_seq || !a->tok_pos || !a->block_ptrs || !a->cu_blocks || !a->qn) { *why = "window attention: bad arguments"; return 0; }
     if (a->heads <= 0 || a->kv_heads <= 0 || a->heads % a->kv_heads || a->dim <= 0 || a->vdim <= 0 || a->block_len <= 0 || a->window < 0 ||
         a->chunk < 0 || (a->talk_scores && !a->talk) || !(a->q_temp_every >= 0.0)) {
         *why = "window attention: heads must be a multiple of kv_heads, sizes positive";
+        return 0;
+    }
+    if (a->maps < 0 || a->maps > 2 || a->keep_first < 0 || (a->maps == 2 && a->talk) || (a->keep_first && !a->window) || a->ld_y < 0) {
+        *why = "window attention: one or two maps (two: without talk), kept first tokens only with a window";
         return 0;
     }
     return 1;
@@ -1172,7 +1185,8 @@ B200H_API int b200h_window_prep(const b200h_window_args* a)
     if (a->n == 0) return 0;
     cudaStream_t st = (cudaStream_t)a->stream;
     B200H_DISPATCH_T(a->dtype, window_prep_kernel<T><<<a->n, 256, 0, st>>>(
-        (const T*)a->q, (const T*)a->k, (const T*)a->v, a->ld, a->heads * a->dim, a->kv_heads * a->dim, a->kv_heads * a->vdim,
+        (const T*)a->q, (const T*)a->k, (const T*)a->v, a->ld, a->heads * window_maps(a) * a->dim, a->kv_heads * window_maps(a) * a->dim,
+        a->kv_heads * a->vdim,
         (const float*)a->bias, (const float*)a->q_norm, (const float*)a->k_norm, a->eps, (const int*)a->tok_seq, (const int*)a->tok_pos,
         (const int64_t*)a->block_ptrs, (const int*)a->cu_blocks, a->layer_off, a->v_off, a->block_len, a->q_temp_coef, a->q_temp_every,
         (float*)a->qn));
@@ -1185,6 +1199,7 @@ B200H_API int b200h_head_rope_prep(const b200h_window_args* a, const b200h_rotar
     if (!window_args_ok(a, &why)) return fail(B200H_ERR_INVALID_ARG, why);
     if (!a->q || !a->k || !a->v || !r || r->pairs < 0 || 2 * r->pairs > a->dim || (r->pairs && !r->freqs))
         return fail(B200H_ERR_INVALID_ARG, "head_rope_prep: bad arguments (2 * rot.pairs <= dim)");
+    if (window_maps(a) > 1) return fail(B200H_ERR_UNSUPPORTED, "head_rope_prep: one map per head");
     if (a->n == 0) return 0;
     cudaStream_t st = (cudaStream_t)a->stream;
     const Rotary rot = make_rotary(r);
@@ -1203,10 +1218,10 @@ B200H_API int b200h_head_rope_prep(const b200h_window_args* a, const b200h_rotar
 
 static size_t window_pv_smem(const b200h_window_args* a, int rows, int tile)
 {
-    const size_t H = a->heads, rh = (size_t)rows * H;
+    const size_t H = a->heads, rh = (size_t)rows * H, rm = rh * window_maps(a);
     auto pad4 = [](size_t v) { return (v + 3) & ~(size_t)3; };
     const bool talk = a->talk && !a->talk_scores;           // pass 2 recombines weights only when the scores were not mixed before it
-    return (size_t)tile * sizeof(char*) + sizeof(float) * (2 * pad4(rh) + (talk ? pad4(H * H) : 0) + (size_t)(talk ? 2 : 1) * rh * tile + rh * a->vdim);
+    return (size_t)tile * sizeof(char*) + sizeof(float) * (2 * pad4(rm) + (talk ? pad4(H * H) : 0) + (size_t)(talk ? 2 : 1) * rh * tile + rh * a->vdim);
 }
 
 struct WindowLaunch {
@@ -1221,11 +1236,11 @@ static void launch_window_kernels(const b200h_window_args* a, const WindowGeom& 
         cudaFuncSetAttribute(window_stats_kernel<T, VEC, NP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)l.stats_smem);
     if (l.pv_smem > 48 * 1024)
         cudaFuncSetAttribute(window_pv_kernel<T, CW, NP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)l.pv_smem);
-    window_stats_kernel<T, VEC, NP><<<dim3(l.blocks, a->kv_heads, a->splits), l.stats_threads, l.stats_smem, st>>>((const float*)a->qn, g,
+    window_stats_kernel<T, VEC, NP><<<dim3(l.blocks, a->kv_heads * g.maps, a->splits), l.stats_threads, l.stats_smem, st>>>((const float*)a->qn, g,
                                                                                                                    (float*)a->ml);
     if (a->talk_scores) {
         // between the passes: the scores of all heads of a row are mixed in place and their maxima and denominators recomputed
-        const int H = a->heads;
+        const int H = a->heads;                  // one map per head (window_args_ok)
         int tile = 128;
         while (tile > 8 && (size_t)H * (H + tile) * sizeof(float) > 96 * 1024) tile /= 2;
         const size_t smem = (size_t)H * (H + tile) * sizeof(float);
@@ -1248,7 +1263,7 @@ static int launch_window_attention(const b200h_window_args* a, WindowGeom g, cud
     while (window_pv_smem(a, g.rows, g.tile) > budget && g.rows > 1) g.rows /= 2;
     WindowLaunch l;
     // pass 1: a thread per key of the range, at most 128
-    const int span = a->window > 0 && a->chunk > 0 ? (a->window < a->chunk ? a->window : a->chunk) : (a->window > 0 ? a->window : a->chunk);
+    const int span = a->window > 0 && a->chunk > 0 ? (a->window < a->chunk ? a->window : a->chunk) : (a->window > 0 ? a->window + a->keep_first : a->chunk);
     const int keys = span > 0 ? span + g.rows - 1 : 1 << 30, per = (keys + a->splits - 1) / a->splits;
     l.stats_threads = per <= 32 ? 32 : (per <= 64 ? 64 : 128);
     auto stats_smem = [&]() { return (size_t)g.rows * rep * a->dim * sizeof(float) + (VEC ? (size_t)l.stats_threads * (a->dim * sizeof(T) + 16) : 0); };
@@ -1262,8 +1277,15 @@ static int launch_window_attention(const b200h_window_args* a, WindowGeom g, cud
     if (pairs <= 2) launch_window_kernels<T, VEC, CW, 2>(a, g, l, st);
     else if (pairs <= 4) launch_window_kernels<T, VEC, CW, 4>(a, g, l, st);
     else launch_window_kernels<T, VEC, CW, 8>(a, g, l, st);
-    window_out_kernel<T><<<dim3(a->n, (H * a->vdim + 255) / 256), 256, 0, st>>>((const float*)a->o_part, a->splits, H * a->vdim, (const T*)a->gate,
-                                                                                a->ld_gate, a->gate_heads ? a->vdim : 1, (T*)a->y);
+    const float scale = a->out_scale;
+    const int64_t ld_y = a->ld_y ? a->ld_y : (int64_t)H * a->vdim;
+    if (a->out_norm)
+        window_out_norm_kernel<T><<<dim3(a->n, H), a->vdim <= 32 ? 32 : (a->vdim <= 64 ? 64 : 128), (size_t)a->vdim * sizeof(float), st>>>(
+            (const float*)a->o_part, a->splits, H * a->vdim, a->vdim, (const T*)a->gate, a->ld_gate, a->gate_heads ? a->vdim : 1, scale, a->eps,
+            (T*)a->y, ld_y);
+    else
+        window_out_kernel<T><<<dim3(a->n, (H * a->vdim + 255) / 256), 256, 0, st>>>((const float*)a->o_part, a->splits, H * a->vdim, (const T*)a->gate,
+                                                                                    a->ld_gate, a->gate_heads ? a->vdim : 1, scale, (T*)a->y, ld_y);
     return 0;
 }
 
@@ -1272,7 +1294,7 @@ B200H_API int b200h_window_attention(const b200h_window_args* a)
     const char* why = "";
     if (!window_args_ok(a, &why)) return fail(B200H_ERR_INVALID_ARG, why);
     if (!a->scores || a->score_ld < 1) return fail(B200H_ERR_INVALID_ARG, "window_attention: no score scratch");
-    if (!a->ml || !a->o_part || !a->y || a->splits < 1 || a->splits > 65535 || a->kv_heads > 65535 || (a->r1 && !a->r2))
+    if (!a->ml || !a->o_part || !a->y || a->splits < 1 || a->splits > 65535 || a->kv_heads > 32767 || a->heads > 65535 || (a->out_norm && a->vdim > 8192) || (a->r1 && !a->r2))
         return fail(B200H_ERR_INVALID_ARG, "window_attention: bad arguments");
     if (a->n == 0) return 0;
     WindowGeom g;
@@ -1280,6 +1302,7 @@ B200H_API int b200h_window_attention(const b200h_window_args* a)
     g.heads = a->heads; g.kv_heads = a->kv_heads; g.dim = a->dim; g.vdim = a->vdim; g.block_len = a->block_len;
     g.window = a->window; g.splits = a->splits; g.scale = a->scale; g.softcap = a->softcap; g.chunk = a->chunk;
     // talk mixes the softmax WEIGHTS inside pass 2, or (talk_scores) the SCORES between the passes: pass 2 then sees no talk
+    g.maps = window_maps(a); g.keep = a->window > 0 ? a->keep_first : 0; g.lambda = a->lambda;
     g.r1 = (const float*)a->r1; g.r2 = (const float*)a->r2; g.talk = a->talk_scores ? nullptr : (const float*)a->talk;
     g.sink = (const float*)a->sink;
     g.tok_seq = (const int*)a->tok_seq; g.tok_pos = (const int*)a->tok_pos;
@@ -1381,8 +1404,8 @@ B200H_API int b200h_conv_rope_prep(const b200h_conv_prep_args* a)
         !a->cu_blocks || a->heads <= 0 || a->kv_heads <= 0 || a->dim <= 0 || a->block_len <= 0 || a->batch <= 0)
         return fail(B200H_ERR_INVALID_ARG, "conv_rope_prep: bad arguments");
     if (a->taps < 1 || a->taps > B200H_MAX_TAPS) return fail(B200H_ERR_UNSUPPORTED, "conv_rope_prep: taps 1..16");
-    if (a->rot.pairs < 0 || 2 * a->rot.pairs > a->dim || (a->rot.pairs && !a->rot.freqs))
-        return fail(B200H_ERR_INVALID_ARG, "conv_rope_prep: rotated pairs do not fit a head");
+    if (a->rot.pairs < 0 || 2 * a->rot.pairs > a->dim || (a->rot.pairs && !a->rot.freqs) || a->rot.halves)
+        return fail(B200H_ERR_INVALID_ARG, "conv_rope_prep: rotated (interleaved) pairs do not fit a head");
     if (a->n == 0) return 0;
     const int channels = (a->heads + a->kv_heads) * a->dim;
     const size_t smem = (size_t)(channels + 2 * a->rot.pairs) * sizeof(float);
@@ -1496,25 +1519,32 @@ B200H_API int b200h_channel_decay_scan(const void* r, const void* k, const void*
     return launched("channel_decay_scan");
 }
 
-B200H_API int b200h_group_norm_gate(const void* o, const void* w, const void* gate, int64_t ld_gate, int n, int count, int groups, int act,
-                                    float eps, void* y, int dtype, void* stream)
+B200H_API int b200h_group_norm_gate_rows(const void* o, const void* w, const void* gate, int64_t ld_gate, int n, int count, int groups, int act,
+                                         float eps, void* y, int64_t ld_y, int dtype, void* stream)
 {
-    if (!o || !w || !gate || !y || count <= 0 || groups <= 0 || count % groups || act < 0 || act > 1)
+    if (!o || !gate || !y || count <= 0 || groups <= 0 || count % groups || act < 0 || act > 1 || ld_y < count)
         return fail(B200H_ERR_INVALID_ARG, "group_norm_gate: bad arguments");
     if (n == 0) return 0;
     cudaStream_t st = (cudaStream_t)stream;
     const int gw = count / groups;
 #define B200H_GNG(NV)                                                                                                                      \
     group_norm_gate_warp_kernel<T, NV><<<n, groups >= 8 ? 256 : 32 * groups, 0, st>>>((const float*)o, (const float*)w, (const T*)gate, ld_gate, \
-                                                                                     count, groups, act, eps, (T*)y)
+                                                                                     count, groups, act, eps, (T*)y, ld_y)
     if (gw <= 256) {            // a warp per group
         B200H_DISPATCH_T(dtype, if (gw <= 32) B200H_GNG(1); else if (gw <= 64) B200H_GNG(2); else if (gw <= 128) B200H_GNG(4); else B200H_GNG(8));
         return launched("group_norm_gate");
     }
 #undef B200H_GNG
     B200H_DISPATCH_T(dtype, group_norm_gate_kernel<T><<<dim3(n, groups), 128, 0, st>>>((const float*)o, (const float*)w, (const T*)gate, ld_gate,
-                                                                                      count, groups, act, eps, (T*)y));
+                                                                                      count, groups, act, eps, (T*)y, ld_y));
     return launched("group_norm_gate");
+}
+
+B200H_API int b200h_group_norm_gate(const void* o, const void* w, const void* gate, int64_t ld_gate, int n, int count, int groups, int act,
+                                    float eps, void* y, int dtype, void* stream)
+{
+    if (!w) return fail(B200H_ERR_INVALID_ARG, "group_norm_gate: bad arguments");
+    return b200h_group_norm_gate_rows(o, w, gate, ld_gate, n, count, groups, act, eps, y, count, dtype, stream);
 }
 
 B200H_API int b200h_xielu(void* x, int64_t count, const void* params, int dtype, void* stream)
@@ -1590,26 +1620,28 @@ B200H_API int b200h_normed_residual_norm(void* x, const void* left, const void* 
     return launched("normed_residual_norm");
 }
 
-B200H_API int b200h_silu_mul_rows(const void* gu, int n, int cols, void* out, int dtype, void* stream)
+B200H_API int b200h_gate_mul_rows(const void* gu, int n, int cols, int act, void* out, int dtype, void* stream)
 {
-    if (!gu || !out || n < 0 || cols <= 0) return fail(B200H_ERR_INVALID_ARG, "silu_mul_rows: bad arguments");
+    if (!gu || !out || n < 0 || cols <= 0 || act < 0 || act > 1) return fail(B200H_ERR_INVALID_ARG, "gate_mul_rows: bad arguments");
     if (n == 0) return 0;
     cudaStream_t st = (cudaStream_t)stream;
     const int64_t count = (int64_t)n * cols;
-    if (cols % 4 == 0 && ((reinterpret_cast<uintptr_t>(gu) | reinterpret_cast<uintptr_t>(out)) & 15) == 0) {
-        B200H_DISPATCH_T(dtype, (silu_mul_rows_kernel<T, 4><<<(unsigned)((count / 4 + 255) / 256), 256, 0, st>>>((const T*)gu, cols, count, (T*)out)));
-    } else {
-        B200H_DISPATCH_T(dtype, (silu_mul_rows_kernel<T, 1><<<(unsigned)((count + 255) / 256), 256, 0, st>>>((const T*)gu, cols, count, (T*)out)));
-    }
-    return launched("silu_mul_rows");
+    const bool vec = cols % 4 == 0 && ((reinterpret_cast<uintptr_t>(gu) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
+#define B200H_GMR(V, GELU) gate_mul_rows_kernel<T, V, GELU><<<(unsigned)((count / V + 255) / 256), 256, 0, st>>>((const T*)gu, cols, count, (T*)out)
+    B200H_DISPATCH_T(dtype, if (vec && act) B200H_GMR(4, true); else if (vec) B200H_GMR(4, false); else if (act) B200H_GMR(1, true); else B200H_GMR(1, false));
+#undef B200H_GMR
+    return launched("gate_mul_rows");
+}
+
+B200H_API int b200h_silu_mul_rows(const void* gu, int n, int cols, void* out, int dtype, void* stream)
+{
+    return b200h_gate_mul_rows(gu, n, cols, 0, out, dtype, stream);
 }
 
 // ------------------------------------------------------------------------------------------------ recurrences with token-dependent gates
-B200H_API int b200h_low_rank_decay(const void* low, int64_t ld, const void* a, const void* bias, int n, int channels, int rank, float tau,
-                                   void* decay, int dtype, void* stream)
+static int low_rank_decay(const void* low, int64_t ld, const void* a, const void* bias, int n, int channels, int rank, float inv_tau,
+                          const void* rate, int dim, void* decay, int dtype, void* stream)
 {
-    if (!low || !a || !bias || !decay || n < 0 || channels <= 0 || rank <= 0 || !(tau > 0.f))
-        return fail(B200H_ERR_INVALID_ARG, "low_rank_decay: bad arguments");
     if (rank > 8192) return fail(B200H_ERR_UNSUPPORTED, "low_rank_decay: rank <= 8192");
     if (n == 0) return 0;
     cudaStream_t st = (cudaStream_t)stream;
@@ -1618,10 +1650,26 @@ B200H_API int b200h_low_rank_decay(const void* low, int64_t ld, const void* a, c
     const bool many = (int64_t)cb * n >= 16 * 296 && rank <= 512;
 #define B200H_LRD(ROWS, V)                                                                                                            \
     low_rank_decay_kernel<T, ROWS, V><<<dim3(cb, (n + ROWS - 1) / ROWS), 128, (size_t)rank * ROWS * sizeof(float), st>>>(              \
-        (const T*)low, ld, (const T*)a, (const float*)bias, n, channels, rank, 1.0f / tau, (float*)decay)
+        (const T*)low, ld, (const T*)a, (const float*)bias, n, channels, rank, inv_tau, (const float*)rate, dim, (float*)decay)
     B200H_DISPATCH_T(dtype, if (many && v == 2) B200H_LRD(16, 2); else if (many) B200H_LRD(16, 1); else if (v == 2) B200H_LRD(1, 2); else B200H_LRD(1, 1));
 #undef B200H_LRD
     return launched("low_rank_decay");
+}
+
+B200H_API int b200h_low_rank_decay(const void* low, int64_t ld, const void* a, const void* bias, int n, int channels, int rank, float tau,
+                                   void* decay, int dtype, void* stream)
+{
+    if (!low || !a || !bias || !decay || n < 0 || channels <= 0 || rank <= 0 || !(tau > 0.f))
+        return fail(B200H_ERR_INVALID_ARG, "low_rank_decay: bad arguments");
+    return low_rank_decay(low, ld, a, bias, n, channels, rank, 1.0f / tau, nullptr, 1, decay, dtype, stream);
+}
+
+B200H_API int b200h_low_rank_rate_decay(const void* low, int64_t ld, const void* a, const void* bias, const void* rate, int n, int heads, int dim,
+                                        int rank, void* decay, int dtype, void* stream)
+{
+    if (!low || !a || !bias || !rate || !decay || n < 0 || heads <= 0 || dim <= 0 || rank <= 0)
+        return fail(B200H_ERR_INVALID_ARG, "low_rank_rate_decay: bad arguments");
+    return low_rank_decay(low, ld, a, bias, n, heads * dim, rank, 1.0f, rate, dim, decay, dtype, stream);
 }
 
 B200H_API int b200h_gated_linear_scan(const void* q, const void* k, const void* v, int64_t ld, float q_scale, const void* decay, void* state,
@@ -1695,4 +1743,175 @@ B200H_API int b200h_real_gated_scan(const b200h_rglru_args* a)
             g, (const T*)a->x, (const T*)a->y, (const T*)a->u, (T*)a->out)));
     }
     return launched("real_gated_scan");
+}
+
+// ------------------------------------------------------------------------------------------------ retention, gated delta rule
+B200H_API int b200h_retention_prep(const void* q, const void* k, int64_t ld, int n, int heads, int dim, float k_scale, const b200h_rotary* r,
+                                   const void* tok_pos, void* qk, int dtype, void* stream)
+{
+    if (!q || !k || !r || !tok_pos || !qk || n < 0 || heads <= 0 || dim <= 0 || r->pairs < 0 || 2 * r->pairs > dim || (r->pairs && !r->freqs))
+        return fail(B200H_ERR_INVALID_ARG, "retention_prep: bad arguments (2 * rot.pairs <= dim)");
+    if (r->pairs > 4096) return fail(B200H_ERR_UNSUPPORTED, "retention_prep: at most 4096 rotated pairs");
+    if (n == 0) return 0;
+    cudaStream_t st = (cudaStream_t)stream;
+    const Rotary rot = make_rotary(r);
+    B200H_DISPATCH_T(dtype, retention_prep_kernel<T><<<n, 256, 2 * (size_t)rot.pairs * sizeof(float), st>>>(
+        (const T*)q, (const T*)k, ld, heads, dim, k_scale, rot, (const int*)tok_pos, (float*)qk));
+    return launched("retention_prep");
+}
+
+template <typename T, bool DELTA>
+static void launch_head_scan(const HeadScan& g, const void* v, int batch, cudaStream_t st)
+{
+    const int ne = (g.dim + 31) / 32;
+#define B200H_HS(NE, NC)                                                                                                             \
+    do {                                                                                                                            \
+        const size_t smem = 2 * (size_t)8 * ((DELTA ? 3 : 2) * NE * 32 + (DELTA ? 2 : 0)) * sizeof(float);                          \
+        if (smem > 48 * 1024)                                                                                                       \
+            cudaFuncSetAttribute(head_scan_kernel<T, DELTA, NE, NC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);       \
+        head_scan_kernel<T, DELTA, NE, NC><<<dim3(g.heads * ((g.vdim + 16 * NC - 1) / (16 * NC)), batch), dim3(32, 4), smem, st>>>( \
+            g, DELTA ? nullptr : (const T*)v, DELTA ? (const float*)v : nullptr);                                                   \
+    } while (0)
+    if (ne <= 1) B200H_HS(1, 2);
+    else if (ne <= 2) B200H_HS(2, 2);
+    else if (ne <= 4) B200H_HS(4, 2);
+    else B200H_HS(8, 1);
+#undef B200H_HS
+}
+
+B200H_API int b200h_retention_scan(const void* qk, const void* v, int64_t ld_v, const void* decay, void* state, int64_t slot_stride, const void* cu_q,
+                                   const void* seq_slot, int batch, int heads, int dim, int vdim, void* out, int dtype, void* stream)
+{
+    if (!qk || !v || !decay || !state || !cu_q || !seq_slot || !out || batch <= 0 || heads <= 0 || dim <= 0 || vdim <= 0)
+        return fail(B200H_ERR_INVALID_ARG, "retention_scan: bad arguments");
+    if (dim > 256 || batch > 65535) return fail(B200H_ERR_UNSUPPORTED, "retention_scan: dim <= 256, batch <= 65535");
+    HeadScan g = {};
+    g.q = (const float*)qk; g.k = g.q + (size_t)heads * dim; g.ld_qk = 2 * (int64_t)heads * dim; g.ld_v = ld_v;
+    g.decay = (const float*)decay; g.state = (float*)state; g.slot_stride = slot_stride;
+    g.cu_q = (const int*)cu_q; g.seq_slot = (const int*)seq_slot;
+    g.heads = g.kv_heads = heads; g.dim = dim; g.vdim = vdim; g.out = (float*)out;
+    g.aligned = dim % 4 == 0 && (reinterpret_cast<uintptr_t>(qk) & 15) == 0;
+    cudaStream_t st = (cudaStream_t)stream;
+    B200H_DISPATCH_T(dtype, (launch_head_scan<T, false>(g, v, batch, st)));
+    return launched("retention_scan");
+}
+
+static bool delta_args_ok(const b200h_delta_args* a)
+{
+    return a && a->u && a->conv_state && a->tok_seq && a->cu_q && a->seq_slot && a->qkv && a->kq && a->beta && a->n >= 0 && a->batch > 0 &&
+           a->heads > 0 && a->kv_heads > 0 && a->heads % a->kv_heads == 0 && a->dim > 0 && a->vdim > 0;
+}
+
+template <typename T>
+static void launch_delta_prep(const b200h_delta_args* a, const DeltaPrep& d, cudaStream_t st)
+{
+    const bool vec = a->dim % 2 == 0 && (a->heads * a->vdim) % 2 == 0 && a->ld % 2 == 0 && reinterpret_cast<uintptr_t>(a->u) % (2 * sizeof(T)) == 0 &&
+                     reinterpret_cast<uintptr_t>(a->conv) % 8 == 0 && reinterpret_cast<uintptr_t>(a->qkv) % 8 == 0;
+    const int v = vec ? 2 : 1, yb = a->kv_heads + (a->heads * a->vdim + 128 * v - 1) / (128 * v);
+    const bool many = (int64_t)yb * a->n >= 8 * 1184 && a->taps <= 4;       // eight rows per block once that leaves eight blocks per SM
+#define B200H_DP(TAPS, ROWS, V)                                                                                                     \
+    delta_prep_kernel<T, TAPS, ROWS, V><<<dim3((a->n + ROWS - 1) / ROWS, yb), 128, (size_t)ROWS * 2 * a->dim * sizeof(float), st>>>( \
+        (const T*)a->u, (const T*)a->b, a->ld, d)
+#define B200H_DP_V(TAPS, ROWS) do { if (vec) B200H_DP(TAPS, ROWS, 2); else B200H_DP(TAPS, ROWS, 1); } while (0)
+    if (a->taps <= 4) { if (many) B200H_DP_V(4, 8); else B200H_DP_V(4, 1); }
+    else B200H_DP_V(B200H_MAX_TAPS, 1);
+#undef B200H_DP_V
+#undef B200H_DP
+}
+
+B200H_API int b200h_delta_prep(const b200h_delta_args* a)
+{
+    if (!delta_args_ok(a) || !a->b || !a->conv) return fail(B200H_ERR_INVALID_ARG, "delta_prep: bad arguments");
+    if (a->taps < 1 || a->taps > B200H_MAX_TAPS || a->dim > 512) return fail(B200H_ERR_UNSUPPORTED, "delta_prep: taps 1..16, dim <= 512");
+    if ((int64_t)a->kv_heads + (int64_t)a->heads * a->vdim / 128 > 65000) return fail(B200H_ERR_UNSUPPORTED, "delta_prep: too many channels");
+    if (a->n == 0) return 0;
+    DeltaPrep d;
+    d.w = (const float*)a->conv; d.taps = a->taps; d.state = (const float*)a->conv_state; d.slot_stride = a->slot_stride;
+    d.tok_seq = (const int*)a->tok_seq; d.cu_q = (const int*)a->cu_q; d.seq_slot = (const int*)a->seq_slot;
+    d.n = a->n; d.heads = a->heads; d.kv_heads = a->kv_heads; d.dim = a->dim; d.vdim = a->vdim;
+    d.q_scale = a->q_scale; d.unit_eps = a->unit_eps;
+    d.qkv = (float*)a->qkv; d.kq = (float*)a->kq; d.beta = (float*)a->beta;
+    cudaStream_t st = (cudaStream_t)a->stream;
+    B200H_DISPATCH_T(a->dtype, launch_delta_prep<T>(a, d, st));
+    return launched("delta_prep");
+}
+
+B200H_API int b200h_delta_scan(const b200h_delta_args* a)
+{
+    if (!delta_args_ok(a) || !a->decay || !a->state || !a->out) return fail(B200H_ERR_INVALID_ARG, "delta_scan: bad arguments");
+    if (a->taps < 1 || a->taps > B200H_MAX_TAPS || a->dim > 256 || a->batch > 65535)
+        return fail(B200H_ERR_UNSUPPORTED, "delta_scan: taps 1..16, dim <= 256, batch <= 65535");
+    if (a->n == 0) return 0;
+    const int KD = a->kv_heads * a->dim;
+    HeadScan g = {};
+    g.channels = 2 * KD + a->heads * a->vdim; g.taps = a->taps;
+    g.q = (const float*)a->qkv; g.k = g.q + KD; g.ld_qk = g.ld_v = g.channels;
+    g.decay = (const float*)a->decay; g.beta = (const float*)a->beta; g.kq = (const float*)a->kq;
+    g.state = (float*)a->state; g.slot_stride = a->slot_stride; g.cu_q = (const int*)a->cu_q; g.seq_slot = (const int*)a->seq_slot;
+    g.heads = a->heads; g.kv_heads = a->kv_heads; g.dim = a->dim; g.vdim = a->vdim; g.out = (float*)a->out;
+    g.aligned = a->dim % 4 == 0 && g.channels % 4 == 0 && ((reinterpret_cast<uintptr_t>(a->qkv) | reinterpret_cast<uintptr_t>(a->decay)) & 15) == 0;
+    g.u = a->u; g.ld_u = a->ld; g.conv_state = (float*)a->conv_state;
+    cudaStream_t st = (cudaStream_t)a->stream;
+    B200H_DISPATCH_T(a->dtype, (launch_head_scan<T, true>(g, g.q + 2 * KD, a->batch, st)));
+    return launched("delta_scan");
+}
+
+// ------------------------------------------------------------------------------------------------ blocks of parallel residual streams
+static bool aligned16(std::initializer_list<const void*> ptrs)
+{
+    for (const void* p : ptrs)
+        if (reinterpret_cast<uintptr_t>(p) & 15) return false;
+    return true;
+}
+
+B200H_API int b200h_embed_streams(const void* tokens, const void* table, float scale, const void* w_embed, void* x, int streams, const void* read,
+                                  const void* w_next, int n, int width, float eps, void* h, int dtype, void* stream)
+{
+    if (!tokens || !table || !x || !read || !w_next || !h || n < 0 || width <= 0 || streams < 1) return fail(B200H_ERR_INVALID_ARG, "embed_streams: bad arguments");
+    const size_t smem = (size_t)width * sizeof(float);
+    if (smem > 200 * 1024) return fail(B200H_ERR_UNSUPPORTED, "embed_streams: a row exceeds shared memory");
+    if (n == 0) return 0;
+    cudaStream_t st = (cudaStream_t)stream;
+    const bool vec = width % 4 == 0 && aligned16({table, w_embed, x, w_next, h});
+#define B200H_ES(V)                                                                                                                    \
+    do {                                                                                                                              \
+        if (smem > 48 * 1024) cudaFuncSetAttribute(embed_streams_kernel<T, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+        embed_streams_kernel<T, V><<<n, 256, smem, st>>>((const int*)tokens, (const T*)table, scale, (const float*)w_embed, (float*)x,  \
+                                                         streams, (const float*)read, (const float*)w_next, width, eps, (T*)h);       \
+    } while (0)
+    B200H_DISPATCH_T(dtype, if (vec) B200H_ES(4); else B200H_ES(1));
+#undef B200H_ES
+    return launched("embed_streams");
+}
+
+template <typename T, int S>
+static void launch_join_streams(float* x, const T* y, const StreamJoin& j, int blocks, bool vec, int write, float* u, T* h, cudaStream_t st)
+{
+    const size_t smem = h ? (size_t)j.width * sizeof(float) : 0;
+#define B200H_JS(V)                                                                                                                       \
+    do {                                                                                                                                 \
+        if (smem > 48 * 1024) cudaFuncSetAttribute(join_streams_kernel<T, S, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+        join_streams_kernel<T, S, V><<<blocks, 256, smem, st>>>(x, y, j, write, u, h);                                                   \
+    } while (0)
+    if (vec) B200H_JS(4); else B200H_JS(1);
+#undef B200H_JS
+}
+
+B200H_API int b200h_join_streams(void* x, int streams, const void* y, const void* ls, const void* mix, const void* out, const void* read,
+                                 const void* w_next, const void* rows, int count, int width, float eps, int write, void* u, void* h, int dtype,
+                                 void* stream)
+{
+    if (!x || count < 0 || width <= 0 || streams < 1 || (y && (!mix || !out)) || (h && !w_next)) return fail(B200H_ERR_INVALID_ARG, "join_streams: bad arguments");
+    if (streams > kMaxStreams) return fail(B200H_ERR_UNSUPPORTED, "join_streams: at most 8 streams");
+    if (h && (size_t)width * sizeof(float) > 200 * 1024) return fail(B200H_ERR_UNSUPPORTED, "join_streams: a row exceeds shared memory");
+    if (count == 0) return 0;
+    StreamJoin j;
+    j.ls = (const float*)ls; j.mix = (const float*)mix; j.out = (const float*)out; j.read = (const float*)read; j.w_next = (const float*)w_next;
+    j.rows = (const int*)rows; j.width = width; j.eps = eps;
+    cudaStream_t st = (cudaStream_t)stream;
+    const bool vec = width % 4 == 0 && aligned16({x, y, ls, w_next, u, h});
+#define B200H_JSS(S) case S: launch_join_streams<T, S>((float*)x, (const T*)y, j, count, vec, write, (float*)u, (T*)h, st); break
+    B200H_DISPATCH_T(dtype, switch (streams) { B200H_JSS(1); B200H_JSS(2); B200H_JSS(3); B200H_JSS(4); B200H_JSS(5); B200H_JSS(6); B200H_JSS(7); B200H_JSS(8); });
+#undef B200H_JSS
+    return launched("join_streams");
 }

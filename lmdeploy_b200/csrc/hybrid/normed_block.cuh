@@ -137,9 +137,9 @@ __global__ void __launch_bounds__(256) normed_residual_norm_kernel(float* __rest
     }
 }
 
-// out[t, i] = silu(gu[t, i]) * gu[t, cols + i]: gu T [n, 2 * cols].  V values per thread.
-template <typename T, int V>
-__global__ void __launch_bounds__(256) silu_mul_rows_kernel(const T* __restrict__ gu, int cols, int64_t count, T* __restrict__ out)
+// out[t, i] = act(gu[t, i]) * gu[t, cols + i]: gu T [n, 2 * cols]; act silu, or GELU: the tanh form of gelu.  V values per thread.
+template <typename T, int V, bool GELU>
+__global__ void __launch_bounds__(256) gate_mul_rows_kernel(const T* __restrict__ gu, int cols, int64_t count, T* __restrict__ out)
 {
     const int64_t i = ((int64_t)blockIdx.x * blockDim.x + threadIdx.x) * V;
     if (i >= count) return;
@@ -150,6 +150,6 @@ __global__ void __launch_bounds__(256) silu_mul_rows_kernel(const T* __restrict_
     load_row<V>(row + c, a);
     load_row<V>(row + cols + c, b);
 #pragma unroll
-    for (int e = 0; e < V; ++e) a[e] = silu_f(a[e]) * b[e];
+    for (int e = 0; e < V; ++e) a[e] = (GELU ? gelu_tanh_f(a[e]) : silu_f(a[e])) * b[e];
     store_row<V>(out + i, a);
 }

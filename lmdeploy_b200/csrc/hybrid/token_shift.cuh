@@ -274,10 +274,10 @@ __global__ void __launch_bounds__(512) channel_decay_scan_kernel(const T* __rest
 }
 
 // y[t] = unit_rms_per_group(o[t]) * w * act(gate[t]) as T: the norm comes before the gate; `groups` equal parts of `count` columns;
-// act 0: sigmoid, 1: silu.
+// act 0: sigmoid, 1: silu; w == nullptr: one; rows of y lie ld_y apart.
 template <typename T>
 __global__ void group_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ w, const T* __restrict__ gate, int64_t ld_gate,
-                                       int count, int groups, int act, float eps, T* __restrict__ y)
+                                       int count, int groups, int act, float eps, T* __restrict__ y, int64_t ld_y)
 {
     __shared__ float red[32];
     const int t = blockIdx.x, g = blockIdx.y, gw = count / groups;
@@ -288,7 +288,7 @@ __global__ void group_norm_gate_kernel(const float* __restrict__ o, const float*
     const float r = 1.0f / sqrtf(ss / (float)gw + eps);
     for (int i = threadIdx.x; i < gw; i += blockDim.x) {
         const float z = to_f(gate[(size_t)t * ld_gate + (size_t)g * gw + i]);
-        y[(size_t)t * count + (size_t)g * gw + i] = from_f<T>(ot[i] * r * w[(size_t)g * gw + i] * (act ? silu_f(z) : sigmoid_f(z)));
+        y[(size_t)t * ld_y + (size_t)g * gw + i] = from_f<T>(ot[i] * r * (w ? w[(size_t)g * gw + i] : 1.0f) * (act ? silu_f(z) : sigmoid_f(z)));
     }
 }
 
@@ -298,7 +298,7 @@ __global__ void group_norm_gate_kernel(const float* __restrict__ o, const float*
 template <typename T, int NV>
 __global__ void __launch_bounds__(256) group_norm_gate_warp_kernel(const float* __restrict__ o, const float* __restrict__ w,
                                                                   const T* __restrict__ gate, int64_t ld_gate, int count, int groups, int act,
-                                                                  float eps, T* __restrict__ y)
+                                                                  float eps, T* __restrict__ y, int64_t ld_y)
 {
     const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5, gw = count / groups;
     for (int g = warp; g < groups; g += nw) {
@@ -314,7 +314,7 @@ __global__ void __launch_bounds__(256) group_norm_gate_warp_kernel(const float* 
             const int c = i * 32 + lane;
             if (c < gw) {
                 const float z = to_f(gate[(size_t)t * ld_gate + at + c]);
-                y[(size_t)t * count + at + c] = from_f<T>(v[i] * r * w[at + c] * (act ? silu_f(z) : sigmoid_f(z)));
+                y[(size_t)t * ld_y + at + c] = from_f<T>(v[i] * r * (w ? w[at + c] : 1.0f) * (act ? silu_f(z) : sigmoid_f(z)));
             }
         }
     }

@@ -1,21 +1,27 @@
 // Kernels of pre-norm hybrid blocks: table rows added to the stream, residual add fused with an RMS norm, softmax attention
 // with grouped key/value heads over a sliding window or within chunks of a paged cache (capped scores, a logarithmic distance
 // penalty, the heads' weight rows recombined by a matrix after the softmax or their scores before it, a sink, an output gate per
-// column or per head), the preparation of an attention that norms per head and rotates, and the squared-relu activation.
+// column or per head, first tokens that a sliding window keeps, two subtracted maps per head), the preparation of an attention that
+// norms per head and rotates, and the squared-relu activation.
 // Included by hybrid_ops.cu inside namespace b200h, after its helpers (to_f / from_f / block_sum / sigmoid_f).
 //
 // Cache entry of position p of a sequence, inside its page (page address + layer_off): the normed key as T at
-// [p % block_len][kv_heads * dim], and, v_off bytes further, the value as T at [p % block_len][kv_heads * vdim].
+// [p % block_len][kv_heads * maps * dim], and, v_off bytes further, the value as T at [p % block_len][kv_heads * vdim].
 //
 // Attention runs in two passes over a row's visible keys [window_first(pos), pos] -- the window's first key, or the first key of
-// the row's chunk --, both cut into `splits` equal key ranges so that a step of few rows still fills the SMs:
+// the row's chunk --, with the sequence's first `keep` positions in front of them where a window keeps those; both passes cut the
+// visible keys, counted without the gap behind the kept ones, into `splits` equal ranges so that a step of few rows still fills the SMs:
 //   pass 1 (window_stats_kernel, one block per row block, key/value head and range): scores of the heads that share the key/value
 //          head, written to a scratch [row, head, key - first visible key], and their running maximum and denominator;
 //   pass 2 (window_pv_kernel, one block per row block and range): the ranges' (maximum, denominator) pairs are merged per head, the
 //          scores of ALL heads of the row are read back, turned into final softmax weights, recombined across heads
 //          (weight'_h = sum_g talk[h, g] weight_g -- this couples every head of a row, hence one block for all of them) and
 //          applied to the values of each head's own key/value head;
-//   window_out_kernel sums the ranges' partial outputs, applies sigmoid(gate) and writes T.
+//   window_out_kernel sums the ranges' partial outputs, applies sigmoid(gate) and writes T (window_out_norm_kernel divides every head
+//          by its root mean square first).
+// An attention of several MAPS per head (differential attention: 2) has maps queries and keys per head, laid out head by head, over one
+// value: pass 1 treats every (head, map) as a head of its own, pass 2 weights a value with w_1 - lambda w_2 -- the maps' outputs are
+// linear in their weights, so the value sum is taken once.
 // A design that mixes the heads' SCORES runs window_mix_scores_kernel between the passes (scores mixed in place, maxima and
 // denominators recomputed from the mixed scores) and pass 2 without its recombination.
 // A block takes `rows` consecutive rows of the step; those of one sequence (consecutive positions) walk their keys together, so a
@@ -120,7 +126,10 @@ __global__ void window_prep_kernel(const T* __restrict__ q, const T* __restrict_
 }
 
 struct WindowGeom {
-    int n, heads, kv_heads, dim, vdim, block_len, window, splits;
+    int n, heads, kv_heads, dim, vdim, block_len, window, splits;       // heads, kv_heads: of the outputs and the values
+    int maps;                 // query and key heads per output / value head (1 or 2)
+    int keep;                 // with a window: the first `keep` positions of the sequence stay visible
+    float lambda;             // maps 2: factor on the second map
     int chunk;                // > 0: a row sees only the keys of its own chunk of this many positions, counted from position 0
     int rows;                 // rows of the step per block (consecutive rows; a block walks the keys once for those of one sequence)
     int tile;                 // keys per tile of pass 2, a multiple of 4, at most 256
@@ -134,7 +143,7 @@ struct WindowGeom {
     const int64_t* block_ptrs;
     const int* cu_blocks;
     int64_t layer_off, v_off;
-    float* scores;            // [rows of the step, heads, score_ld]: score of a row's key j at index j - (the row's first visible key)
+    float* scores;            // [rows of the step, heads * maps, score_ld]: score of a row's i-th visible key at index i
     int score_ld;
 };
 
@@ -145,19 +154,38 @@ __device__ __forceinline__ int window_first(const WindowGeom& g, int pos)
     return g.chunk > 0 ? max(lo, pos / g.chunk * g.chunk) : lo;
 }
 
-// The key range `z` of consecutive rows of one sequence at positions first .. last: [j0, j1).  Every row masks the keys of the
-// range that it does not see.
-__device__ __forceinline__ void window_range(const WindowGeom& g, int first, int last, int z, int& j0, int& j1)
+// how many kept positions lie in front of the keys [lo, ...)
+__device__ __forceinline__ int window_kept(const WindowGeom& g, int lo) { return min(g.keep, lo); }
+
+// Visible keys of consecutive rows of one sequence at positions first .. last, taken together: kept positions 0 .. kept - 1, then
+// lo .. last.  Range `z` of them is [i0, i1) of this list.  Every row masks the keys of the range that it does not see.
+struct WindowKeys {
+    int lo, kept, i0, i1;
+    __device__ __forceinline__ int at(int i) const { return i < kept ? i : i - kept + lo; }
+};
+
+__device__ __forceinline__ WindowKeys window_range(const WindowGeom& g, int first, int last, int z)
 {
-    const int lo = window_first(g, first);
-    const int per = (last - lo + g.splits) / g.splits;         // ceil((last - lo + 1) / splits)
-    j0 = lo + z * per;
-    j1 = min(last + 1, j0 + per);
+    WindowKeys w;
+    w.lo = window_first(g, first);
+    w.kept = window_kept(g, w.lo);
+    const int count = w.kept + last - w.lo + 1, per = (count + g.splits - 1) / g.splits;
+    w.i0 = z * per;
+    w.i1 = min(count, w.i0 + per);
+    return w;
 }
 
 __device__ __forceinline__ bool window_sees(const WindowGeom& g, int pos, int j)
 {
-    return j <= pos && j >= window_first(g, pos);
+    const int lo = window_first(g, pos);
+    return j <= pos && (j >= lo || j < window_kept(g, lo));
+}
+
+// place of key j in the list of keys that the row at position pos sees
+__device__ __forceinline__ int window_index(const WindowGeom& g, int pos, int j)
+{
+    const int lo = window_first(g, pos);
+    return j >= lo ? j - lo + window_kept(g, lo) : j;
 }
 
 // score of head `head` for a key at distance `dist` behind the query, from the raw dot product
@@ -224,21 +252,22 @@ __device__ __forceinline__ void merge_ml(float& m, float& l, float om, float ol)
     m = mx;
 }
 
-// Pass 1.  grid (row blocks, kv_heads, splits), up to 128 threads: thread i walks keys j0 + i, j0 + i + blockDim, ... of the range
-// for all (row, head) pairs of the block's rows that belong to one sequence and of the heads that share key/value head blockIdx.y.
+// Pass 1.  grid (row blocks, kv_heads * maps, splits), up to 128 threads: thread i walks the i-th, i + blockDim-th, ... key of the range
+// for all (row, head) pairs of the block's rows that belong to one sequence and of the heads that share key head blockIdx.y.
 template <typename T, bool VEC, int NP>
 __global__ void __launch_bounds__(128) window_stats_kernel(const float* __restrict__ qn, WindowGeom g, float* __restrict__ ml)
 {
     extern __shared__ __align__(16) float win_smem[];
     __shared__ float red_m[4][kMaxPairs], red_l[4][kMaxPairs];
     const int c = blockIdx.y, z = blockIdx.z, tid = threadIdx.x, nw = blockDim.x >> 5;
-    const int H = g.heads, D = g.dim, rep = H / g.kv_heads;
+    const int H = g.heads * g.maps, D = g.dim, rep = g.heads / g.kv_heads;
+    const int h0 = c / g.maps * rep * g.maps + c % g.maps;                   // the heads that share key head c: h0, h0 + maps, ...
     const int t0 = blockIdx.x * g.rows, t1 = min(g.n, t0 + g.rows);
     float* qs = win_smem;                                                    // [rows * rep][dim]
     // VEC: one key row per thread after the queries, rows 16 bytes apart from a multiple of 128 so that the 16-byte reads of a
     // quarter warp fall into different banks
     char* stage = reinterpret_cast<char*>(win_smem + (size_t)g.rows * rep * D) + (size_t)tid * (D * sizeof(T) + 16);
-    const size_t k_row = (size_t)g.kv_heads * D;
+    const size_t k_row = (size_t)g.kv_heads * g.maps * D;
     for (int ta = t0; ta < t1;) {
         const int s = g.tok_seq[ta];
         int tb = ta + 1;
@@ -247,18 +276,18 @@ __global__ void __launch_bounds__(128) window_stats_kernel(const float* __restri
         __syncthreads();
         for (int i = tid; i < pairs * D; i += blockDim.x) {
             const int u = i / D, d = i - u * D, r = u / rep, hh = u - r * rep;
-            qs[i] = qn[((size_t)(ta + r) * H + c * rep + hh) * D + d];
+            qs[i] = qn[((size_t)(ta + r) * H + h0 + hh * g.maps) * D + d];
         }
         __syncthreads();
-        int j0, j1;
-        window_range(g, pos, pos + nr - 1, z, j0, j1);
+        const WindowKeys keys = window_range(g, pos, pos + nr - 1, z);
         const int64_t* pages = g.block_ptrs + g.cu_blocks[s];
         for (int ub = 0; ub < pairs; ub += NP) {
             const int cnt = min(NP, pairs - ub);
             float m[NP], l[NP];
 #pragma unroll
             for (int u = 0; u < NP; ++u) { m[u] = -1e30f; l[u] = 0.f; }
-            for (int j = j0 + tid; j < j1; j += blockDim.x) {
+            for (int i = keys.i0 + tid; i < keys.i1; i += blockDim.x) {
+                const int j = keys.at(i);
                 const T* key = reinterpret_cast<const T*>(window_page(g, pages, j)) + (size_t)(j % g.block_len) * k_row + (size_t)c * D;
                 if (VEC) {
                     // the thread's key travels to its own row of shared memory by asynchronous 16-byte copies: all of them are in
@@ -277,8 +306,9 @@ __global__ void __launch_bounds__(128) window_stats_kernel(const float* __restri
                     if (u < cnt) {
                         const int r = (ub + u) / rep, hh = (ub + u) - r * rep;
                         if (window_sees(g, pos + r, j)) {
-                            const float sc = window_score(g, acc[u], c * rep + hh, pos + r - j);
-                            g.scores[((size_t)(ta + r) * H + c * rep + hh) * g.score_ld + (j - window_first(g, pos + r))] = sc;
+                            const int head = h0 + hh * g.maps;
+                            const float sc = window_score(g, acc[u], head, pos + r - j);
+                            g.scores[((size_t)(ta + r) * H + head) * g.score_ld + window_index(g, pos + r, j)] = sc;
                             merge_ml(m[u], l[u], sc, 1.0f);
                         }
                     }
@@ -302,7 +332,7 @@ __global__ void __launch_bounds__(128) window_stats_kernel(const float* __restri
                 float mm = red_m[0][tid], ll = red_l[0][tid];
                 for (int w = 1; w < nw; ++w) merge_ml(mm, ll, red_m[w][tid], red_l[w][tid]);
                 const int r = (ub + tid) / rep, hh = (ub + tid) - r * rep;
-                float* dst = ml + (((size_t)(ta + r) * H + c * rep + hh) * g.splits + z) * 2;
+                float* dst = ml + (((size_t)(ta + r) * H + h0 + hh * g.maps) * g.splits + z) * 2;
                 dst[0] = mm;
                 dst[1] = ll;
             }
@@ -330,7 +360,7 @@ template <> __device__ __forceinline__ void load_cols<bf16, 4>(const bf16* __res
 __device__ __forceinline__ int pad4(int v) { return (v + 3) & ~3; }
 
 // Pass 2.  grid (row blocks, splits), 256 threads.  Shared memory: the tile's value row addresses [tile], then floats
-// mx [rows * heads] | linv [rows * heads] | talk [heads][heads] | p [rows * heads][tile] | p2 [rows * heads][tile] |
+// mx [rows * heads * maps] | linv [rows * heads * maps] | talk [heads][heads] | p [rows * heads][tile] | p2 [rows * heads][tile] |
 // o [rows * heads][vdim] (every part padded to a multiple of four floats).
 // CW: value columns per thread and walk (4: 8- or 16-byte reads of the values).  NP: (row, head) pairs per walk over a value -- 2 for
 // a step of single tokens with two heads per key/value head, which keeps registers low and more blocks resident.
@@ -339,11 +369,11 @@ __global__ void __launch_bounds__(256) window_pv_kernel(WindowGeom g, const floa
 {
     extern __shared__ __align__(16) unsigned char win_raw[];
     const int z = blockIdx.y, tid = threadIdx.x, nt = blockDim.x;
-    const int H = g.heads, G = g.kv_heads, rep = H / G, V = g.vdim, KT = g.tile;
+    const int H = g.heads, G = g.kv_heads, rep = H / G, V = g.vdim, KT = g.tile, HM = H * g.maps;
     const char** vrow = reinterpret_cast<const char**>(win_raw);
     float* mx = reinterpret_cast<float*>(win_raw + (size_t)KT * sizeof(char*));
-    float* linv = mx + pad4(g.rows * H);
-    float* talk = linv + pad4(g.rows * H);
+    float* linv = mx + pad4(g.rows * HM);
+    float* talk = linv + pad4(g.rows * HM);
     float* p = talk + (g.talk ? pad4(H * H) : 0);
     float* p2 = g.talk ? p + (size_t)g.rows * H * KT : p;
     float* o = p2 + (size_t)g.rows * H * KT;
@@ -358,31 +388,34 @@ __global__ void __launch_bounds__(256) window_pv_kernel(WindowGeom g, const floa
         const int nr = tb - ta, pos = g.tok_pos[ta], pairs = nr * rep;
         __syncthreads();
         for (int i = tid; i < nr * H * V; i += nt) o[i] = 0.f;
-        for (int i = tid; i < nr * H; i += nt) {
-            const float* src = ml + ((size_t)ta * H + i) * g.splits * 2;
+        for (int i = tid; i < nr * HM; i += nt) {
+            const float* src = ml + ((size_t)ta * HM + i) * g.splits * 2;
             float mm = src[0], ll = src[1];
             for (int k = 1; k < g.splits; ++k) merge_ml(mm, ll, src[2 * k], src[2 * k + 1]);
-            if (g.sink) merge_ml(mm, ll, g.sink[i % H], 1.0f);
+            if (g.sink) merge_ml(mm, ll, g.sink[i % HM], 1.0f);
             mx[i] = mm;
             linv[i] = 1.0f / ll;
         }
-        int j0, j1;
-        window_range(g, pos, pos + nr - 1, z, j0, j1);
+        const WindowKeys keys = window_range(g, pos, pos + nr - 1, z);
         const int64_t* pages = g.block_ptrs + g.cu_blocks[s];
-        for (int jt = j0; jt < j1; jt += KT) {
-            const int kt = min(KT, j1 - jt), kt4 = pad4(kt);
+        for (int jt = keys.i0; jt < keys.i1; jt += KT) {
+            const int kt = min(KT, keys.i1 - jt), kt4 = pad4(kt);
             __syncthreads();                      // the previous tile's readers are done; mx / o of this segment are in place
             for (int jj = tid; jj < kt; jj += nt) {
-                const int j = jt + jj;
+                const int j = keys.at(jt + jj);
                 vrow[jj] = window_page(g, pages, j) + g.v_off + (size_t)(j % g.block_len) * v_row;
             }
             // final softmax weights of every (row, head) for the tile's keys (zero for a key the row does not see and for the
             // keys that pad the tile to a multiple of four), from the scores pass 1 left
             for (int item = tid; item < nr * H * kt4; item += nt) {
-                const int rh = item / kt4, jj = item - rh * kt4, j = jt + jj, r = rh / H;
+                const int rh = item / kt4, jj = item - rh * kt4, j = keys.at(jt + jj), r = rh / H;
                 float w = 0.f;
-                if (jj < kt && window_sees(g, pos + r, j))
-                    w = expf(g.scores[((size_t)ta * H + rh) * g.score_ld + (j - window_first(g, pos + r))] - mx[rh]) * linv[rh];
+                if (jj < kt && window_sees(g, pos + r, j)) {
+                    const int first = rh * g.maps;
+                    const float* sc = g.scores + ((size_t)ta * HM + first) * g.score_ld + window_index(g, pos + r, j);
+                    w = expf(sc[0] - mx[first]) * linv[first];
+                    if (g.maps == 2) w -= g.lambda * (expf(sc[g.score_ld] - mx[first + 1]) * linv[first + 1]);
+                }
                 p[(size_t)rh * KT + jj] = w;
             }
             __syncthreads();
@@ -460,10 +493,11 @@ __global__ void __launch_bounds__(256) window_pv_kernel(WindowGeom g, const floa
     }
 }
 
-// y[t, i] = (sum over ranges of o_part[t, z, i]) * sigmoid(gate[t, i / gate_div]) as T (gate_div 1: a gate per column; vdim: one per head)
+// y[t, i] = (sum over ranges of o_part[t, z, i]) * scale * sigmoid(gate[t, i / gate_div]) as T (gate_div 1: a gate per column; vdim: one
+// per head); rows of y lie ld_y apart
 template <typename T>
 __global__ void window_out_kernel(const float* __restrict__ o_part, int splits, int cols, const T* __restrict__ gate, int64_t ld_gate,
-                                  int gate_div, T* __restrict__ y)
+                                  int gate_div, float scale, T* __restrict__ y, int64_t ld_y)
 {
     const int t = blockIdx.x, i = blockIdx.y * blockDim.x + threadIdx.x;          // one column per thread
     if (i >= cols) return;
@@ -472,7 +506,34 @@ __global__ void window_out_kernel(const float* __restrict__ o_part, int splits, 
 #pragma unroll 8
     for (int z = 0; z < splits; ++z) a += src[(size_t)z * cols];
     if (gate) a *= sigmoid_f(to_f(gate[(size_t)t * ld_gate + i / gate_div]));
-    y[(size_t)t * cols + i] = from_f<T>(a);
+    y[(size_t)t * ld_y + i] = from_f<T>(a * scale);
+}
+
+// The same with every head divided by its root mean square over vdim first: one block per (row, head); a thread sums the ranges of its
+// columns once and keeps them in shared memory [vdim].
+template <typename T>
+__global__ void window_out_norm_kernel(const float* __restrict__ o_part, int splits, int cols, int vdim, const T* __restrict__ gate,
+                                       int64_t ld_gate, int gate_div, float scale, float eps, T* __restrict__ y, int64_t ld_y)
+{
+    extern __shared__ __align__(16) float won_smem[];
+    __shared__ float red[32];
+    const int t = blockIdx.x, at = blockIdx.y * vdim;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < vdim; i += blockDim.x) {
+        const float* src = o_part + (size_t)t * splits * cols + at + i;
+        float a = 0.f;
+#pragma unroll 8
+        for (int z = 0; z < splits; ++z) a += src[(size_t)z * cols];
+        won_smem[i] = a;
+        ss = fmaf(a, a, ss);
+    }
+    ss = block_sum(ss, red);
+    const float r = scale / sqrtf(ss / (float)vdim + eps);
+    for (int i = threadIdx.x; i < vdim; i += blockDim.x) {
+        float a = won_smem[i] * r;                            // written above by this same thread
+        if (gate) a *= sigmoid_f(to_f(gate[(size_t)t * ld_gate + (at + i) / gate_div]));
+        y[(size_t)t * ld_y + at + i] = from_f<T>(a);
+    }
 }
 
 // Scores mixed ACROSS heads before the softmax: for every row and visible key, s'_h = sum_g talk[h, g] s_g, in place in the
@@ -484,11 +545,9 @@ __global__ void __launch_bounds__(256) window_mix_scores_kernel(WindowGeom g, co
 {
     extern __shared__ __align__(16) float mix_smem[];
     const int t = blockIdx.x, z = blockIdx.y, H = g.heads, tid = threadIdx.x, nt = blockDim.x;
-    const int pos = g.tok_pos[t], lo = window_first(g, pos);
-    int j0, j1;
-    window_range(g, pos, pos, z, j0, j1);
-    j0 -= lo;                                                 // the scratch is indexed from the row's first visible key
-    j1 -= lo;
+    const int pos = g.tok_pos[t];
+    const WindowKeys keys = window_range(g, pos, pos, z);     // the scratch is indexed like the row's list of visible keys
+    const int j0 = keys.i0, j1 = keys.i1;
     float* tk = mix_smem;
     float* raw = mix_smem + H * H;
     float* row = g.scores + (size_t)t * H * g.score_ld;
@@ -526,7 +585,7 @@ __global__ void __launch_bounds__(256) window_mix_scores_kernel(WindowGeom g, co
 //   1. the projections' biases are added (float);
 //   2. every head of q and of k is divided by its root mean square over `dim` and multiplied by a weight of `dim` entries that all
 //      heads share (wq / wk; nullptr: no norm of that projection);
-//   3. pairs (2i, 2i+1), i < rot.pairs, of every head turn by position * freqs[i];
+//   3. pairs (2i, 2i+1) -- or, rot.halves, (i, i + rot.pairs) --, i < rot.pairs, of every head turn by position * freqs[i];
 //   4. queries, times query_growth -> qn (float), keys and (biased) values -> the row's cache entry as T.
 // Shared memory: (heads + kv_heads) * dim floats, then 2 * rot.pairs floats of cos / sin.
 template <typename T>
@@ -573,6 +632,16 @@ __global__ void head_rope_prep_kernel(const T* __restrict__ q, const T* __restri
         }
         __syncwarp();
         // one lane per pair of dimensions; a turning pair is whole (2 * rot.pairs <= dim), the rest pass unchanged
+        if (rot.halves) {
+            for (int d = lane; d < dim; d += 32) {
+                float a = x[d];
+                if (d < rot.pairs) a = a * cs[d] - x[d + rot.pairs] * sn[d];
+                else if (d < 2 * rot.pairs) a = a * cs[d - rot.pairs] + x[d - rot.pairs] * sn[d - rot.pairs];
+                if (h < heads) qn[(size_t)t * HD + (size_t)h * dim + d] = a * growth;
+                else k_dst[(size_t)(h - heads) * dim + d] = from_f<T>(a);
+            }
+            continue;
+        }
         for (int d = 2 * lane; d < dim; d += 64) {
             const bool two = d + 1 < dim;
             float a = x[d], b = two ? x[d + 1] : 0.f;

@@ -6,8 +6,9 @@ A hybrid decoder mixes layer kinds, so a sequence owns two things between steps:
     windowed-, chunked- or convolved-rotary-attention layer its normed (and rotated) keys and its values (as T);
   * one slot of the StatePool (handed out by scheduler.Scheduler's slot list) -- per layer the last taps-1 inputs of the
     short convolution (of both sublayers in pre-norm blocks; of the stacked q | k projection of a convolved attention; of the
-    x | B | C channels of a state-space mixer; of the biased convolution branch of an RG-LRU), per decayed-linear-attention,
-    channel-decay or gated-linear layer the [heads, vdim, dim] float state, per state-space layer the [heads, vdim, state] float
+    x | B | C channels of a state-space mixer; of the biased convolution branch of an RG-LRU; of the q | k | v channels of a gated
+    delta rule), per decayed-linear-attention,
+    channel-decay, gated-linear, retention or gated-delta layer the [heads, vdim, dim] float state, per state-space layer the [heads, vdim, state] float
     state and per RG-LRU one float per channel; in shared-norm blocks per run the last normed row and the
     last shifted row (the token shift), and once the id of the last token (hashed bigram embedding).
 A layer that a spec loops (HybridSpec.loop) is executed several times per step with the same weights: caches and states
@@ -83,7 +84,9 @@ class HybridModel:
         self.cache_off, self.rot_off, self.conv_off, self.mix_off, self.conv2_off, self.v_off = {}, {}, {}, {}, {}, {}
         self.shift_off = {}
         self.runs = spec.runs()
-        if spec.block not in ("post_norm", "pre_norm", "parallel", "shared_norm", "sandwich"):
+        if spec.streams != 1 and (spec.block != "streams" or not 1 <= spec.streams <= H.MAX_STREAMS):
+            raise NotImplementedError(f"{spec.streams} residual streams (1..{H.MAX_STREAMS}, in stream blocks)")
+        if spec.block not in ("post_norm", "pre_norm", "parallel", "shared_norm", "sandwich", "streams"):
             raise NotImplementedError(f"block {spec.block!r}")
         pre = spec.block == "pre_norm"
         page = slot = 0
@@ -99,7 +102,7 @@ class HybridModel:
             if spec.block == "shared_norm":     # token shift: the last normed row and the last shifted row
                 self.shift_off[r] = slot
                 slot += 2 * spec.width
-            elif spec.block not in ("parallel", "sandwich"):
+            elif spec.block not in ("parallel", "sandwich", "streams"):
                 slot += (taps - 1) * spec.width
             if pre and layer.mlp is not None:
                 self.conv2_off[r] = slot
@@ -137,21 +140,35 @@ class HybridModel:
                 slot += m.heads * m.vdim * m.dim
             elif m.kind in ("window_attention", "paired"):
                 if m.kind == "paired":
-                    if m.left.kind != "window_attention" or (spec.block, m.right.kind) not in (("shared_norm", "channel_decay"), ("sandwich", "gated_linear")):
-                        raise NotImplementedError("paired mixers: windowed attention beside a channel-decay recurrence in shared-norm blocks "
-                                                  "or beside gated linear attention in sandwich blocks")
+                    if m.left.kind != "window_attention" or (spec.block, m.right.kind) not in (("shared_norm", "channel_decay"), ("sandwich", "gated_linear"),
+                                                                                               ("streams", "gated_delta")):
+                        raise NotImplementedError("paired mixers: windowed attention beside a channel-decay recurrence in shared-norm blocks, "
+                                                  "beside gated linear attention in sandwich blocks or beside a gated delta rule in stream blocks")
                     if m.right.dim > 256:
-                        raise NotImplementedError("channel-decay recurrence, gated linear attention: dim <= 256")
+                        raise NotImplementedError("channel-decay recurrence, gated linear attention, gated delta rule: dim <= 256")
+                    if m.right.kind == "gated_delta":
+                        if not 1 <= m.right.conv_taps <= H.MAX_TAPS:
+                            raise NotImplementedError(f"conv taps {m.right.conv_taps} (1..{H.MAX_TAPS})")
+                        self.conv_off[r] = slot
+                        slot += (m.right.conv_taps - 1) * m.right.conv_channels
                     slot = _align(slot, 4)                  # 16-byte reads of the state's columns
                     self.mix_off[r] = slot
                     slot += m.right.heads * m.right.vdim * m.right.dim
                     m = m.left
                 if m.window and m.chunk:
                     raise NotImplementedError("windowed attention: a sliding window or chunks, not both")
-                # in a region [block_len, kv_heads * dim] keys as T then [block_len, kv_heads * vdim] values as T
+                if m.keep_first and not m.window or m.maps not in (1, 2):
+                    raise NotImplementedError("windowed attention: kept first tokens only with a sliding window, one or two maps per head")
+                # in a region [block_len, kv_heads * maps * dim] keys as T then [block_len, kv_heads * vdim] values as T
                 self.cache_off[r] = page
-                self.v_off[r] = _align(block_len * m.kv_heads * m.dim * esize)
-                page += self.v_off[r] + _align(block_len * m.kv_heads * m.vdim * esize)
+                self.v_off[r] = _align(block_len * m.k_cols * esize)
+                page += self.v_off[r] + _align(block_len * m.v_cols * esize)
+            elif m.kind == "retention":
+                if m.dim > 256:
+                    raise NotImplementedError("retention: dim <= 256")
+                slot = _align(slot, 4)                      # 16-byte reads of the state's columns
+                self.mix_off[r] = slot
+                slot += m.heads * m.vdim * m.dim
             elif m.kind == "rglru":
                 if not 1 <= m.conv_taps <= H.MAX_TAPS:
                     raise NotImplementedError(f"conv taps {m.conv_taps} (1..{H.MAX_TAPS})")
@@ -163,7 +180,7 @@ class HybridModel:
                 raise NotImplementedError(m.kind)
         self.block_bytes = max(page, 16)
         self.layer_bytes = self.block_bytes         # bytes of one block per "layer unit" as the engine sizes pools: whole block
-        self.slot_floats = slot
+        self.slot_floats = _align(slot, 4) if spec.block == "streams" else slot
         self.w = {}
         self.weight_bytes = 0
         self.grouped_experts_rows = 24    # steps that give an expert this many rows on average run the experts as grouped GEMMs
@@ -208,19 +225,18 @@ class HybridModel:
 
         W = s.width
         pre = s.block == "pre_norm"
-        par = s.block == "parallel"
+        par, strm = s.block == "parallel", s.block == "streams"
 
         def norm_w(name):
-            # pre-norm and parallel blocks store a norm weight as its deviation from one: the kernels get the full factor
+            # pre-norm, parallel and stream blocks store a norm weight as its deviation from one: the kernels get the full factor
             t = f32(name, (W,))
-            return t + 1.0 if (pre or par) and not s.plain_norms else t
+            return t + 1.0 if (pre or par or strm) and not s.plain_norms else t
 
         def window_weights(p, ck, m):
             """Windowed attention: checkpoint tensors ck + 'q' ... -> w[p + 'in'] ..."""
-            HD, GD, GV, HV = m.heads * m.dim, m.kv_heads * m.dim, m.kv_heads * m.vdim, m.heads * m.vdim
-            gate_cols = (m.heads if m.gate_per_head else HV) if m.gate else 0
+            HD, GD, GV, HV = m.q_cols, m.k_cols, m.v_cols, m.heads * m.vdim
             parts = [ck + "q", ck + "k", ck + "v"] + ([ck + "g"] if m.gate else [])
-            w[p + "in"] = lin(*parts, shape=(HD + GD + GV + gate_cols, W))
+            w[p + "in"] = lin(*parts, shape=(m.proj_cols, W))
             if m.bias:          # added in float by the kernel that norms q and k and stores the cache (no bias pass over the GEMM's output)
                 w[p + "in.b"] = torch.cat([f32(ck + f"{k}.b", (cols,)) for k, cols in (("q", HD), ("k", GD), ("v", GV))]).contiguous()
             w[p + "o"] = lin(ck + "o", shape=(W, HV))
@@ -235,13 +251,29 @@ class HybridModel:
             if m.sink:
                 w[p + "sink"] = f32(ck + "sink", (m.heads,))
             if m.rot is not None:
-                freqs, mag = m.rot.frequencies()
-                w[p + "freqs"] = torch.tensor(freqs, dtype=torch.float64, device=dev)
-                w[p + "mag"] = float(mag)
+                rotation(p, m.rot)
+            if m.maps == 2:     # one number per layer, the same for every token
+                l1, k1, l2, k2 = (get(ck + k).to(torch.float64) for k in ("lq1", "lk1", "lq2", "lk2"))
+                for t in (l1, k1, l2, k2):
+                    if tuple(t.shape) != (m.dim,):
+                        raise ValueError(f"{ck}lq1..lk2: shape {tuple(t.shape)}, expected {(m.dim,)}")
+                w[p + "lambda"] = float(torch.exp((l1 * k1).sum()) - torch.exp((l2 * k2).sum()) + m.diff)
+
+        def rotation(p, rot):
+            freqs, mag = rot.frequencies()
+            w[p + "freqs"] = torch.tensor(freqs, dtype=torch.float64, device=dev)
+            w[p + "mag"] = float(mag)
+
+        def padded(rows, to=8):
+            """A stacked matrix with zero rows up to a multiple of `to`: what follows it stays aligned."""
+            pad = -rows.shape[0] % to
+            return torch.cat([rows, rows.new_zeros(pad, rows.shape[1])]) if pad else rows
 
         w["embed"] = lin("embed", shape=(s.vocab, W))
         w["head"] = w["embed"] if s.tied_head else lin("head", shape=(s.vocab, W))
         w["final.norm"] = norm_w("final.norm") * s.logit_scale          # the head is linear in it: scaling the norm scales the logits
+        if strm:
+            w["embed.norm"] = norm_w("embed.norm")
         if s.bigram is not None:
             w["bigram"] = lin("bigram", shape=(s.bigram.buckets + 1, W))
         if s.max_positions:
@@ -252,7 +284,12 @@ class HybridModel:
             p, m = f"l{i}.", layer.mixer
             w[p + "norm1"] = norm_w(p + "norm1")
             shared, both_ends = s.block == "shared_norm", s.block == "sandwich"
-            if shared:
+            if strm:
+                for q in (1, 2) if layer.mlp is not None else (1,):
+                    w[p + f"ls{q}"] = f32(p + f"ls{q}", (W,))
+                    for k, shape in (("in", (s.streams,)), ("out", (s.streams,)), ("mix", (s.streams, s.streams))):
+                        w[p + f"hc{q}.{k}"] = f32(p + f"hc{q}.{k}", shape)
+            elif shared:
                 w[p + "shift"] = f32(p + "shift", (W,))
             elif both_ends:
                 w[p + "norm1b"] = norm_w(p + "norm1b")
@@ -305,6 +342,34 @@ class HybridModel:
                 for k in ("ra.b", "ri.b"):
                     w[p + k] = f32(p + "mix." + k, (m.blocks, size)).reshape(R)
                 w[p + "o"] = lin(p + "mix.o", shape=(W, R))
+            elif m.kind == "retention":
+                HD, HV = m.heads * m.dim, m.heads * m.vdim
+                w[p + "in"] = lin(p + "mix.q", p + "mix.k", p + "mix.v", p + "mix.g", shape=(2 * HD + 2 * HV, W))
+                w[p + "o"] = lin(p + "mix.o", shape=(W, HV))
+                w[p + "decay"] = torch.tensor(m.decay, dtype=torch.float32, device=dev)
+                rotation(p, m.rot)
+            elif m.kind == "paired" and m.right.kind == "gated_delta":
+                window_weights(p + "left.", p + "mix.left.", m.left)
+                R, ck = m.right, p + "mix.right."
+                KD, HD, HV = R.kv_heads * R.dim, R.heads * R.dim, R.heads * R.vdim
+                # both sides read the same rows: ONE product for left q | k | v | g and right q | k | v, a1, g1, b, every part from a multiple
+                # of eight columns on
+                parts = {"left": w.pop(p + "left.in"), "u": lin(ck + "q", ck + "k", ck + "v", shape=(R.conv_channels, W)),
+                         "a1": lin(ck + "a1", shape=(R.decay_rank, W)), "g1": lin(ck + "g1", shape=(R.gate_rank, W)), "b": lin(ck + "b", shape=(R.heads, W))}
+                at, cols = 0, {}
+                for k in parts:
+                    cols[k], parts[k] = at, padded(parts[k])
+                    at += parts[k].shape[0]
+                w[p + "in"], w[p + "cols"] = torch.cat(list(parts.values())).contiguous(), cols
+                w[p + "right.conv"] = torch.cat([f32(ck + f"{k}.conv", (n_, R.conv_taps)) for k, n_ in (("q", KD), ("k", KD), ("v", HV))]).t().contiguous()
+                w[p + "right.a2"] = lin(ck + "a2", shape=(HD, R.decay_rank)).t().contiguous()
+                w[p + "right.dt_bias"] = f32(ck + "dt_bias", (HD,))
+                w[p + "right.rate"] = torch.exp(f32(ck + "A_log", (R.heads,)))
+                w[p + "right.g2"] = lin(ck + "g2", shape=(HV, R.gate_rank))
+                # the sides' scales ride on what is multiplied in float anyway; one output product takes both sides' columns
+                w[p + "right.norm"] = f32(ck + "norm", (R.vdim,)).repeat(R.heads) * m.scales[1]
+                o = torch.cat([w.pop(p + "left.o"), lin(ck + "o", shape=(W, HV))], 1)
+                w[p + "o"] = padded(o.t()).t().contiguous()
             elif m.kind == "paired" and m.right.kind == "gated_linear":
                 window_weights(p + "left.", p + "mix.left.", m.left)
                 R, ck = m.right, p + "mix.right."
@@ -348,7 +413,7 @@ class HybridModel:
                 if pre:
                     w[p + "canon2"] = f32(p + "canon2", (W, s.conv_taps))
                 if f.kind == "dense":
-                    if f.act == "silu_gate":
+                    if f.act in H.MLP_GATE_ACT:
                         w[p + "up"] = lin(p + "mlp.gate", p + "mlp.up", shape=(2 * f.ff, W))
                     else:
                         w[p + "up"] = lin(p + "mlp.up", shape=(f.ff, W))
@@ -378,7 +443,7 @@ class HybridModel:
 
         def get(name):
             shape = self.tensor_shapes()[name]
-            if name.endswith(("norm1", "norm2", "final.norm")) and self.spec.block in ("pre_norm", "parallel") and not self.spec.plain_norms:
+            if name.endswith(("norm1", "norm2", "final.norm", "embed.norm")) and self.spec.block in ("pre_norm", "parallel", "streams") and not self.spec.plain_norms:
                 return 0.1 * torch.randn(shape, generator=g)            # stored as the deviation from one
             if name.endswith((".conv", ".conv.b")):
                 return torch.randn(shape, generator=g) / (shape[-1] if name.endswith(".conv") else 10.0)
@@ -388,6 +453,13 @@ class HybridModel:
                 return torch.log(torch.expm1(0.001 + 0.099 * torch.rand(shape, generator=g)))
             if name.endswith(".D"):
                 return torch.ones(shape)
+            if ".hc" in name:                                            # a stream keeps most of itself and takes some of the others
+                own = torch.eye(shape[0]) if len(shape) == 2 else torch.full(shape, 1.0 if name.endswith("out") else 1.0 / shape[0])
+                return own + 0.1 * torch.randn(shape, generator=g) / shape[0]
+            if name.endswith((".ls1", ".ls2")):
+                return 0.5 + 0.1 * torch.randn(shape, generator=g)
+            if name.endswith((".lq1", ".lk1", ".lq2", ".lk2")):
+                return 0.1 * torch.randn(shape, generator=g)
             if name.endswith(("norm1", "norm2", "norm1b", "norm2b", ".norm", ".out")):
                 return 1.0 + 0.1 * torch.randn(shape, generator=g)
             if name.endswith("shift") or ".mu." in name:
@@ -414,7 +486,7 @@ class HybridModel:
                 return torch.softmax(torch.randn(shape, generator=g), 0)
             if name.endswith("sink"):
                 return torch.randn(shape, generator=g)
-            scale = 0.02 if name == "embed" else 1.0 / (shape[-1] ** 0.5)
+            scale = 0.02 if name == "embed" and self.spec.block != "streams" else 1.0 / (shape[-1] ** 0.5)
             return (torch.randn(shape, generator=g) * scale).to(torch.bfloat16)
 
         self.load_weights(get)
@@ -423,8 +495,10 @@ class HybridModel:
         """Checkpoint tensor names -> shapes for this spec."""
         s, W = self.spec, self.spec.width
         pre = s.block == "pre_norm"
-        par = s.block == "parallel"
+        par, strm = s.block == "parallel", s.block == "streams"
         out = {"embed": (s.vocab, W)}
+        if strm:
+            out["embed.norm"] = (W,)
         if not s.tied_head:
             out["head"] = (s.vocab, W)
         out["final.norm"] = (W,)
@@ -437,7 +511,9 @@ class HybridModel:
         shared, both_ends = s.block == "shared_norm", s.block == "sandwich"
 
         def window_shapes(ck, m):
-            HD, GD, GV, HV = m.heads * m.dim, m.kv_heads * m.dim, m.kv_heads * m.vdim, m.heads * m.vdim
+            HD, GD, GV, HV = m.q_cols, m.k_cols, m.v_cols, m.heads * m.vdim
+            if m.maps == 2:
+                out.update({ck + k: (m.dim,) for k in ("lq1", "lk1", "lq2", "lk2")})
             out.update({ck + "q": (HD, W), ck + "k": (GD, W), ck + "v": (GV, W), ck + "o": (W, HV)})
             if m.bias:
                 out.update({ck + "q.b": (HD,), ck + "k.b": (GD,), ck + "v.b": (GV,)})
@@ -455,7 +531,10 @@ class HybridModel:
         for i, layer in enumerate(s.layers):
             p, m = f"l{i}.", layer.mixer
             out[p + "norm1"] = (W,)
-            if shared:
+            if strm:
+                for q in (1, 2) if layer.mlp is not None else (1,):
+                    out.update({p + f"ls{q}": (W,), p + f"hc{q}.in": (s.streams,), p + f"hc{q}.out": (s.streams,), p + f"hc{q}.mix": (s.streams, s.streams)})
+            elif shared:
                 out[p + "shift"] = (W,)
             elif both_ends:
                 out[p + "norm1b"] = (W,)
@@ -485,6 +564,17 @@ class HybridModel:
                 out.update({p + "mix." + k: (R,) for k in ("y.b", "x.b", "conv.b", "lam")})
                 for k in ("ra", "ri"):
                     out.update({p + "mix." + k: (m.blocks, size, size), p + f"mix.{k}.b": (m.blocks, size)})
+            elif m.kind == "retention":
+                HD, HV = m.heads * m.dim, m.heads * m.vdim
+                out.update({p + "mix.q": (HD, W), p + "mix.k": (HD, W), p + "mix.v": (HV, W), p + "mix.g": (HV, W), p + "mix.o": (W, HV)})
+            elif m.kind == "paired" and m.right.kind == "gated_delta":
+                window_shapes(p + "mix.left.", m.left)
+                R, ck = m.right, p + "mix.right."
+                KD, HD, HV = R.kv_heads * R.dim, R.heads * R.dim, R.heads * R.vdim
+                for k, n in (("q", KD), ("k", KD), ("v", HV)):
+                    out.update({ck + k: (n, W), ck + k + ".conv": (n, R.conv_taps)})
+                out.update({ck + "b": (R.heads, W), ck + "A_log": (R.heads,), ck + "norm": (R.vdim,), ck + "a1": (R.decay_rank, W),
+                            ck + "a2": (HD, R.decay_rank), ck + "dt_bias": (HD,), ck + "g1": (R.gate_rank, W), ck + "g2": (HV, R.gate_rank), ck + "o": (W, HV)})
             elif m.kind == "paired" and m.right.kind == "gated_linear":
                 window_shapes(p + "mix.left.", m.left)
                 R, ck = m.right, p + "mix.right."
@@ -512,7 +602,7 @@ class HybridModel:
                 if pre:
                     out[p + "canon2"] = (W, s.conv_taps)
                 if f.kind == "dense":
-                    if f.act == "silu_gate":
+                    if f.act in H.MLP_GATE_ACT:
                         out[p + "mlp.gate"] = (f.ff, W)
                     out.update({p + "mlp.up": (f.ff, W), p + "mlp.down": (W, f.ff)})
                     if f.act == "xielu":
@@ -570,6 +660,10 @@ class HybridModel:
         st = self._stream()
         if s.max_positions and max_pos >= s.max_positions:
             raise ValueError(f"position {max_pos}: the model has {s.max_positions} learned positions")
+        if s.block == "streams":
+            return self._step_streams(n=n, batch=batch, tokens=tokens, tok_seq=tok_seq, tok_pos=tok_pos, cu_q=cu_q, seq_slot=seq_slot,
+                                      block_ptrs=block_ptrs, cu_blocks=cu_blocks, state=state, rows=rows, n_rows=n_rows, max_pos=max_pos,
+                                      trace=trace)
         if s.block == "sandwich":
             return self._step_sandwich(n=n, batch=batch, tokens=tokens, tok_seq=tok_seq, tok_pos=tok_pos, cu_q=cu_q, seq_slot=seq_slot,
                                        block_ptrs=block_ptrs, cu_blocks=cu_blocks, state=state, rows=rows, n_rows=n_rows, max_pos=max_pos,
@@ -859,6 +953,125 @@ class HybridModel:
                                               dt, st), "group_norm_rows")
             return self._logits(xn)
 
+    def _step_streams(self, *, n, batch, tokens, tok_seq, tok_pos, cu_q, seq_slot, block_ptrs, cu_blocks, state, rows, n_rows, max_pos,
+                      trace=None):
+        """The step of stream blocks: the residual is `streams` copies x_s; per sublayer u = sum_s in[s] x_s, y = ls * sublayer(n(u)),
+        x_t <- sum_s mix[s, t] x_s + out[t] * y, all streams at once.  One kernel joins a sublayer's output into the streams and emits
+        the next sublayer's normed input; the last join runs only over the rows whose logits are wanted."""
+        s, lib, w, dev, T, dt = self.spec, self.lib, self.w, self.device, self.T, self.dt
+        W, S, eps, st = s.width, s.streams, s.norm_eps, self._stream()
+        c = StepArrays(n=n, batch=batch, tok_seq=tok_seq, tok_pos=tok_pos, cu_q=cu_q, seq_slot=seq_slot, block_ptrs=block_ptrs,
+                       cu_blocks=cu_blocks, state=state, max_pos=max_pos)
+        x = torch.empty(n, S, W, dtype=torch.float32, device=dev)
+        h = torch.empty(n, W, dtype=T, device=dev)
+        subs = [(r, i, q) for r, (i, _) in enumerate(self.runs) for q in ((1, 2) if s.layers[i].mlp is not None else (1,))]
+        with self.timed("embed"):
+            i, q = subs[0][1:] if subs else (None, None)
+            ones = torch.ones(S, dtype=torch.float32, device=dev) if not subs else None
+            H.check(lib.b200h_embed_streams(tokens.data_ptr(), w["embed"].data_ptr(), s.embedding_scale, w["embed.norm"].data_ptr(), x.data_ptr(), S,
+                                            (w[f"l{i}.hc{q}.in"] if subs else ones).data_ptr(), (w[f"l{i}.norm{q}"] if subs else w["final.norm"]).data_ptr(),
+                                            n, W, eps, h.data_ptr(), dt, st), "embed_streams")
+        y = prev = None                  # the last sublayer's output and its weights' prefix and number
+
+        def join(read, norm, out, count, rows=None, write=1, u=None):
+            i, q = prev if y is not None else (None, None)
+            with self.timed("streams + norm"):
+                H.check(lib.b200h_join_streams(
+                    x.data_ptr(), S, None if y is None else y.data_ptr(), *([None] * 3 if y is None else [w[f"l{i}.{k}"].data_ptr() for k in (
+                        f"ls{q}", f"hc{q}.mix", f"hc{q}.out")]), None if read is None else read.data_ptr(), None if norm is None else norm.data_ptr(),
+                    None if rows is None else rows.data_ptr(), count, W, eps, write, None if u is None else u.data_ptr(),
+                    None if out is None else out.data_ptr(), dt, st), "join_streams")
+
+        for at, (r, i, q) in enumerate(subs):
+            if at > 0:
+                join(w[f"l{i}.hc{q}.in"], w[f"l{i}.norm{q}"], h, n)
+            if q == 1:
+                m = self.paired_delta_mixer(r, i, h, c) if s.layers[i].mixer.kind == "paired" else self.mixer(r, i, h, c)
+                with self.timed("gemm out"):
+                    y = self._linear(m, w[f"l{i}.o"])
+            else:
+                y = self.dense_mlp(i, h)
+            prev = (i, q)
+            if trace is not None and (at + 1 == len(subs) or subs[at + 1][0] != r):
+                total = torch.empty(n, W, dtype=torch.float32, device=dev)
+                join(None, None, None, n, u=total)
+                y = None
+                trace.append(total)
+        xn = torch.empty(n_rows, W, dtype=T, device=dev)
+        join(None, w["final.norm"], xn, n_rows, rows=rows, write=0)
+        with self.timed("head"):
+            return self._logits(xn)
+
+    def paired_delta_mixer(self, r, i, h, c):
+        """Chunked or windowed attention beside a gated delta rule (layer i in run r) over h [n, width] (T): one stacked product feeds both
+        sides, each writes its scaled columns of one matrix, which the output product takes whole.  Returns [n, columns of both] (T)."""
+        m, w, n, p = self.spec.layers[i].mixer, self.w, c.n, f"l{i}."
+        HL, HR = m.left.heads * m.left.vdim, m.right.heads * m.right.vdim
+        with self.timed("gemm in"):
+            proj = self._linear(h, w[p + "in"])
+        cols = w[p + "o"].shape[1]
+        y = (torch.empty if cols == HL + HR else torch.zeros)(n, cols, dtype=self.T, device=self.device)      # padding columns stay zero
+        self.window_mixer(i, None, c, run=r, m=m.left, p=p + "left.", proj=proj, out=y, scale=m.scales[0])
+        self.gated_delta_mixer(i, proj, c, run=r, m=m.right, p=p + "right.", cols=w[p + "cols"], out=y[:, HL:])
+        return y
+
+    def gated_delta_mixer(self, i, proj, c, run, m, p, cols, out):
+        """The gated delta rule of layer i: proj [n, ..] (T) holds its q | k | v, a1, g1 and b columns from cols[..] on.  Convolutions, unit
+        vectors and step sizes; decays; the recurrence on the sequence's float state; then the per-head norm and the low-rank gate, into
+        `out` (T, rows as far apart as the matrix it is a part of)."""
+        w, lib, dev, n, st = self.w, self.lib, self.device, c.n, self._stream()
+        HD, HV = m.heads * m.dim, m.heads * m.vdim
+        ld, es, base = proj.stride(0), proj.element_size(), proj.data_ptr()
+        f32 = dict(dtype=torch.float32, device=dev)
+        a = H.DeltaArgs()
+        a.n, a.batch, a.heads, a.kv_heads, a.dim, a.vdim, a.taps = n, c.batch, m.heads, m.kv_heads, m.dim, m.vdim, m.conv_taps
+        a.q_scale, a.unit_eps = m.dim ** -0.5, m.unit_eps
+        a.u, a.b, a.ld, a.conv = base + es * cols["u"], base + es * cols["b"], ld, w[p + "conv"].data_ptr()
+        a.conv_state, a.state, a.slot_stride = c.state.ptr(self.conv_off[run]), c.state.ptr(self.mix_off[run]), c.state.storage.stride(0)
+        qkv, kq, beta = torch.empty(n, m.conv_channels, **f32), torch.empty(n, m.kv_heads, **f32), torch.empty(n, m.heads, **f32)
+        decay, o = torch.empty(n, HD, **f32), torch.empty(n, HV, **f32)
+        a.qkv, a.kq, a.beta, a.decay, a.out = qkv.data_ptr(), kq.data_ptr(), beta.data_ptr(), decay.data_ptr(), o.data_ptr()
+        a.tok_seq, a.cu_q, a.seq_slot, a.dtype, a.stream = c.tok_seq.data_ptr(), c.cu_q.data_ptr(), c.seq_slot.data_ptr(), self.dt, st
+        with self.timed("short convs + unit vectors"):
+            H.check(lib.b200h_delta_prep(C.byref(a)), "delta_prep")
+        with self.timed("low-rank decay"):
+            H.check(lib.b200h_low_rank_rate_decay(base + es * cols["a1"], ld, w[p + "a2"].data_ptr(), w[p + "dt_bias"].data_ptr(),
+                                                  w[p + "rate"].data_ptr(), n, m.heads, m.dim, m.decay_rank, decay.data_ptr(), self.dt, st),
+                    "low_rank_rate_decay")
+        with self.timed("gated delta rule"):
+            H.check(lib.b200h_delta_scan(C.byref(a)), "delta_scan")
+        with self.timed("gemm gate"):
+            gate = self._linear(proj[:, cols["g1"]:cols["g1"] + m.gate_rank], w[p + "g2"])
+        with self.timed("head norm + gate"):
+            H.check(lib.b200h_group_norm_gate_rows(o.data_ptr(), w[p + "norm"].data_ptr(), gate.data_ptr(), gate.stride(0), n, HV, m.heads,
+                                                   H.GATE_ACT["sigmoid"], self.spec.norm_eps, out.data_ptr(), out.stride(0), self.dt, st),
+                    "group_norm_gate")
+
+    def retention_mixer(self, i, h, c, run=None):
+        """Retention of layer i over h [n, width] (T): one stacked projection (q | k | v | gate), rotation of q and k, the per-head
+        recurrence on the sequence's float state, then the unit norm per head times silu(gate).  Returns [n, heads * vdim] (T)."""
+        m, w, lib, dev, n, st = self.spec.layers[i].mixer, self.w, self.lib, self.device, c.n, self._stream()
+        p = f"l{i}."
+        HD, HV = m.heads * m.dim, m.heads * m.vdim
+        with self.timed("gemm in"):
+            proj = self._linear(h, w[p + "in"])
+        ld, es, base = proj.stride(0), proj.element_size(), proj.data_ptr()
+        qk = torch.empty(n, 2 * HD, dtype=torch.float32, device=dev)
+        rot = H.Rotary(w[p + "freqs"].data_ptr(), m.rot.dims // 2, w[p + "mag"], int(m.rot.halves))
+        with self.timed("rotate q, k"):
+            H.check(lib.b200h_retention_prep(base, base + es * HD, ld, n, m.heads, m.dim, m.dim ** -0.5, C.byref(rot), c.tok_pos.data_ptr(),
+                                             qk.data_ptr(), self.dt, st), "retention_prep")
+        o = torch.empty(n, HV, dtype=torch.float32, device=dev)
+        with self.timed("retention"):
+            H.check(lib.b200h_retention_scan(qk.data_ptr(), base + es * 2 * HD, ld, w[p + "decay"].data_ptr(),
+                                             c.state.ptr(self.mix_off[i if run is None else run]), c.state.storage.stride(0), c.cu_q.data_ptr(),
+                                             c.seq_slot.data_ptr(), c.batch, m.heads, m.dim, m.vdim, o.data_ptr(), self.dt, st), "retention_scan")
+        y = torch.empty(n, HV, dtype=self.T, device=dev)
+        with self.timed("head norm + gate"):
+            H.check(lib.b200h_group_norm_gate_rows(o.data_ptr(), None, base + es * (2 * HD + HV), ld, n, HV, m.heads, H.GATE_ACT["silu"],
+                                                   self.spec.norm_eps, y.data_ptr(), HV, self.dt, st), "group_norm_gate")
+        return y
+
     def gated_linear_mixer(self, i, proj, c, run=None, m=None, p=None):
         """Gated linear attention of layer i over its columns of a stacked projection, proj [n, q | k | v | g | a1] (T): the per-channel
         decays from the low-rank columns, the per-head recurrence on the sequence's float state, then the per-head norm and
@@ -969,6 +1182,8 @@ class HybridModel:
             return self.ssm_mixer(i, h, c, run=r)
         if kind == "rglru":
             return self.rglru_mixer(i, h, c, run=r)
+        if kind == "retention":
+            return self.retention_mixer(i, h, c, run=r)
         return self.decay_mixer(i, h, c, run=r)
 
     def window_splits(self, n, window, max_pos):
@@ -990,16 +1205,17 @@ class HybridModel:
         ld = (keys + 255) // 256 * 256
         return min(ld, (window + 3) // 4 * 4) if window else ld
 
-    def window_mixer(self, i, h, c, run=None, m=None, p=None, proj=None):
+    def window_mixer(self, i, h, c, run=None, m=None, p=None, proj=None, out=None, scale=1.0):
         """Windowed attention of layer i (m, p: the spec and weight prefix of one side of a paired mixer): one stacked projection
-        (q | k | v | gate; proj: its columns of a wider product that the caller has made already); biases + RMS norm of q and k (over their whole projections, or per head followed by a rotation) + cache
+        (q | k | v | gate; proj: a wider product that the caller has made already, these columns first); biases + RMS norm of q and k (over their whole projections, or per head followed by a rotation) + cache
         store in one kernel; then attention over the window or chunk of cached keys with capped scores, distance penalty, the heads'
-        scores or softmax weights recombined, a sink, and the output gate.  Returns [n, heads * vdim] (T)."""
+        scores or softmax weights recombined or two maps subtracted, a sink, a norm per head, and the output gate, times `scale`.  Returns
+        [n, heads * vdim] (T): the first columns of `out` where one is given."""
         r = i if run is None else run
         m = self.spec.layers[i].mixer if m is None else m
         p = f"l{i}." if p is None else p
         w, lib, dev, T, n = self.w, self.lib, self.device, self.T, c.n
-        HD, GD, GV, HV = m.heads * m.dim, m.kv_heads * m.dim, m.kv_heads * m.vdim, m.heads * m.vdim
+        HD, GD, GV, HV = m.q_cols, m.k_cols, m.v_cols, m.heads * m.vdim
         if proj is None:
             with self.timed("gemm in"):
                 proj = self._linear(h, w[p + "in"])
@@ -1010,6 +1226,9 @@ class HybridModel:
         a.chunk, a.talk_scores, a.gate_heads = m.chunk, int(m.talk_scores), int(m.gate_per_head)
         a.splits = self.window_splits(n, m.span, c.max_pos)
         a.scale, a.softcap, a.eps = m.scale, m.softcap, self.spec.norm_eps
+        a.maps, a.keep_first, a.out_scale = m.maps, m.keep_first, scale
+        if m.maps == 2:
+            a.lambda_, a.out_norm, a.out_scale = w[p + "lambda"], 1, scale * (1.0 - m.diff)
         if m.q_temp is not None:
             a.q_temp_coef, a.q_temp_every = m.q_temp
         a.q, a.k, a.v, a.ld = base, base + es * HD, base + es * (HD + GD), ld
@@ -1027,14 +1246,15 @@ class HybridModel:
             a.sink = w[p + "sink"].data_ptr()
         if m.gate:
             a.gate, a.ld_gate = base + es * (HD + GD + GV), ld
-        y = torch.empty(n, HV, dtype=T, device=dev)
+        y = torch.empty(n, HV, dtype=T, device=dev) if out is None else out
+        a.ld_y = y.stride(0)
         a.tok_seq, a.tok_pos = c.tok_seq.data_ptr(), c.tok_pos.data_ptr()
         a.block_ptrs, a.cu_blocks = c.block_ptrs.data_ptr(), c.cu_blocks.data_ptr()
         a.layer_off, a.v_off, a.dtype, a.stream = self.cache_off[r], self.v_off[r], self.dt, self._stream()
         if m.head_norm or m.rot is not None:
             if m.qk_norm and not m.head_norm:
                 raise NotImplementedError("rotation after a norm over the whole projection")
-            rot = H.Rotary(w[p + "freqs"].data_ptr(), m.rot.dims // 2, w[p + "mag"]) if m.rot is not None else H.Rotary(None, 0, 1.0)
+            rot = H.Rotary(w[p + "freqs"].data_ptr(), m.rot.dims // 2, w[p + "mag"], int(m.rot.halves)) if m.rot is not None else H.Rotary(None, 0, 1.0)
             with self.timed("head norm + rotate + cache store"):
                 H.check(lib.b200h_head_rope_prep(C.byref(a), C.byref(rot)), "head_rope_prep")
         else:
@@ -1045,23 +1265,24 @@ class HybridModel:
 
     def _window_attend(self, a, m, c, qn, y, name):
         """The two attention passes over the cache for a prepared step (a: WindowArgs with sizes, switches, cache offsets and, if any,
-        gate filled in; qn float [n, heads * dim]; y T [n, heads * vdim]).  Pass 1 leaves every row's scores in a scratch [rows,
+        gate filled in; qn float [n, heads * maps * dim]; y T, heads * vdim columns).  Pass 1 leaves every row's scores in a scratch [rows,
         heads, keys a row can see] for pass 2; the step's rows go through the two passes in chunks that keep the scratch within
         `window_scratch_bytes`."""
-        n, HD, HV, es = c.n, m.heads * m.dim, m.heads * m.vdim, y.element_size()
+        n, HV, es, heads = c.n, m.heads * m.vdim, y.element_size(), m.heads * getattr(m, "maps", 1)
+        HD, ld_y = heads * m.dim, y.stride(0)
         f32 = dict(dtype=torch.float32, device=self.device)
         a.score_ld = self.window_score_ld(getattr(m, "span", m.window), c.max_pos)
-        chunk = max(4, self.window_scratch_bytes // (4 * m.heads * a.score_ld) // 4 * 4)
+        chunk = max(4, self.window_scratch_bytes // (4 * heads * a.score_ld) // 4 * 4)
         rows = min(n, chunk)
-        scores = torch.empty(rows, m.heads, a.score_ld, **f32)
-        ml = torch.empty(rows, m.heads, a.splits, 2, **f32)
+        scores = torch.empty(rows, heads, a.score_ld, **f32)
+        ml = torch.empty(rows, heads, a.splits, 2, **f32)
         o_part = torch.empty(rows, a.splits, HV, **f32)
         a.scores, a.ml, a.o_part = scores.data_ptr(), ml.data_ptr(), o_part.data_ptr()
         gate, ld_gate = a.gate, a.ld_gate
         with self.timed(name):
             for at in range(0, n, chunk):
                 a.n = min(chunk, n - at)
-                a.qn, a.y = qn.data_ptr() + 4 * at * HD, y.data_ptr() + es * at * HV
+                a.qn, a.y = qn.data_ptr() + 4 * at * HD, y.data_ptr() + es * at * ld_y
                 a.tok_seq, a.tok_pos = c.tok_seq.data_ptr() + 4 * at, c.tok_pos.data_ptr() + 4 * at
                 if gate:
                     a.gate = gate + es * at * ld_gate
@@ -1093,6 +1314,7 @@ class HybridModel:
         a.n, a.heads, a.kv_heads, a.dim, a.vdim, a.block_len, a.window = n, m.heads, m.kv_heads, m.dim, m.vdim, self.block_len, m.window
         a.splits = self.window_splits(n, m.window, c.max_pos)
         a.scale, a.softcap, a.eps = m.scale, 0.0, self.spec.norm_eps
+        a.ld_y = HV
         if m.sink is not None:
             a.sink = w[p + "sink"].data_ptr()
         a.qn = qn.data_ptr()
@@ -1133,22 +1355,22 @@ class HybridModel:
                                               self.spec.norm_eps, y.data_ptr(), self.dt, st), "gate_group_norm")
         return y
 
-    def gated_mlp(self, h, up, down, name="gated feed-forward"):
-        """down(silu(gate h) * up h) over h [n, width] (T) with gate and up stacked in one matrix -> [n, width] (T)."""
+    def gated_mlp(self, h, up, down, name="gated feed-forward", act="silu_gate"):
+        """down(act(gate h) * up h) over h [n, width] (T) with gate and up stacked in one matrix -> [n, width] (T)."""
         with self.timed(f"gemm {name}"):
             gu = self._linear(h, up)
         n, ff = h.shape[0], up.shape[0] // 2
         a = torch.empty(n, ff, dtype=self.T, device=self.device)
-        with self.timed("silu * up"):
-            H.check(self.lib.b200h_silu_mul_rows(gu.data_ptr(), n, ff, a.data_ptr(), self.dt, self._stream()), "silu_mul_rows")
+        with self.timed("act * up"):
+            H.check(self.lib.b200h_gate_mul_rows(gu.data_ptr(), n, ff, H.MLP_GATE_ACT[act], a.data_ptr(), self.dt, self._stream()), "gate_mul_rows")
         with self.timed(f"gemm {name}"):
             return self._linear(a, down)
 
     def dense_mlp(self, i, h):
         """Dense feed-forward of layer i over its input h [n, width] (T): down(act(up h)) -> [n, width] (T)."""
         f, w = self.spec.layers[i].mlp, self.w
-        if f.act == "silu_gate":
-            return self.gated_mlp(h, w[f"l{i}.up"], w[f"l{i}.down"])
+        if f.act in H.MLP_GATE_ACT:
+            return self.gated_mlp(h, w[f"l{i}.up"], w[f"l{i}.down"], act=f.act)
         if f.act not in ("relu2", "xielu"):
             raise NotImplementedError(f"activation {f.act!r}")
         with self.timed("gemm up"):

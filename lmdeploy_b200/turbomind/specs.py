@@ -102,6 +102,7 @@ class RotarySpec:
     base: float
     scaling: tuple = None
     linear: float = 1.0                 # every frequency is divided by this (positions stretched by a constant)
+    halves: bool = False                # dimension i pairs with i + dims/2 instead of 2i with 2i+1
 
     def frequencies(self):
         """-> ([angle per position of pair i], factor on cos and sin), in double precision."""
@@ -150,6 +151,18 @@ class DecayAttentionSpec:
 
 
 @dataclass(frozen=True)
+class RetentionSpec:
+    """Linear attention with a fixed decay per head on rotated queries and keys: S <- decay_h S + k v^T, o = S^T q, k rotated and then
+    divided by sqrt(dim); every head's o is divided by its root mean square (no weight), times silu(W_g h), then projected."""
+    heads: int
+    dim: int
+    vdim: int
+    decay: tuple
+    rot: RotarySpec
+    kind = "retention"
+
+
+@dataclass(frozen=True)
 class WindowAttentionSpec:
     """Softmax attention with grouped key/value heads over a sliding window of cached keys and values, without rotation.
     Score of query i and key j (max(0, i - window + 1) <= j <= i): scale * q.k, capped as softcap * tanh(. / softcap), minus
@@ -180,12 +193,40 @@ class WindowAttentionSpec:
     gate_per_head: bool = False
     # (coef, every): a query at position p is multiplied by 1 + coef * ln(1 + floor((p + 1) / every))
     q_temp: tuple = None
+    keep_first: int = 0           # with a window: the sequence's first keep_first positions stay visible to every row
+    # maps 2: differential attention.  Every head has two queries and every key/value head two keys (projections laid out head by head as
+    # [map 1, map 2]) and one value; a head's output is softmax_1 v - lambda softmax_2 v with lambda = exp(sum(lq1 * lk1)) -
+    # exp(sum(lq2 * lk2)) + diff, one learned number per layer, divided by its root mean square over vdim and multiplied by 1 - diff.
+    maps: int = 1
+    diff: float = 0.0
     kind = "window_attention"
 
     @property
     def span(self):
         """The most keys a row sees (0: all earlier positions)."""
-        return min(self.window, self.chunk) if self.window and self.chunk else (self.window or self.chunk)
+        if self.window and self.chunk:
+            return min(self.window, self.chunk)
+        return self.window + self.keep_first if self.window else self.chunk
+
+    @property
+    def q_cols(self):
+        return self.heads * self.maps * self.dim
+
+    @property
+    def k_cols(self):
+        return self.kv_heads * self.maps * self.dim
+
+    @property
+    def v_cols(self):
+        return self.kv_heads * self.vdim
+
+    @property
+    def gate_cols(self):
+        return (self.heads if self.gate_per_head else self.heads * self.vdim) if self.gate else 0
+
+    @property
+    def proj_cols(self):
+        return self.q_cols + self.k_cols + self.v_cols + self.gate_cols
 
 
 @dataclass(frozen=True)
@@ -279,11 +320,37 @@ class RgLruSpec:
 
 
 @dataclass(frozen=True)
+class GatedDeltaSpec:
+    """Gated delta rule: per head, S a [dim, vdim] float matrix,
+        S <- diag(g_t) S;  u = beta_t (v_t - S^T k_t);  S <- S + k_t u^T;  o = S^T q_t.
+    q and k (kv_heads x dim; head h reads h / (heads / kv_heads)) and v (heads x vdim) each pass a short causal convolution per channel
+    (conv_taps weights, no bias, the last column is the current token's) and silu; q and k become unit vectors per head, q divided by
+    sqrt(dim); beta = sigmoid(W_b h) per head; g = exp(-exp(A_log_h) softplus(A2 (A1 h) + dt_bias)) per head and key channel
+    (inner size decay_rank); every head's o is RMS-normed over vdim with a weight all heads share, times sigmoid(G2 (G1 h)) (inner size
+    gate_rank), then projected."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    conv_taps: int
+    decay_rank: int
+    gate_rank: int
+    unit_eps: float = 1e-6        # unit vectors: x / sqrt(sum(x^2) + unit_eps)
+    kind = "gated_delta"
+
+    @property
+    def conv_channels(self):
+        """Channels of the stacked q | k | v convolution."""
+        return 2 * self.kv_heads * self.dim + self.heads * self.vdim
+
+
+@dataclass(frozen=True)
 class PairedMixerSpec:
     """Two mixers side by side on the same input, each with an output projection of its own; the result is
-    (rms(left) * w_left + rms(right) * w_right) / 2 with RMS norms over the model width."""
+    (rms(left) * w_left + rms(right) * w_right) / 2 with RMS norms over the model width, or, with scales (a, b), a * left + b * right."""
     left: object                        # WindowAttentionSpec
-    right: object                       # ChannelDecaySpec (shared-norm blocks) | GatedLinearSpec (sandwich blocks)
+    right: object                       # ChannelDecaySpec (shared-norm blocks) | GatedLinearSpec (sandwich blocks) | GatedDeltaSpec (stream blocks)
+    scales: tuple = None
     kind = "paired"
 
 
@@ -315,7 +382,7 @@ class RoutedExpertsSpec:
 class DenseMlpSpec:
     """down(act(up h)); act 'relu2' = the square of relu; 'xielu' = softplus(p) z^2 + z / 2 for z > 0 and
     (1/2 + softplus(q)) (exp(z) - 1 - z) + z / 2 otherwise, with the two learned numbers p, q of the layer's 'mlp.act';
-    'silu_gate' = down(silu(gate h) * up h) with a gate matrix beside up."""
+    'silu_gate' = down(silu(gate h) * up h) with a gate matrix beside up; 'gelu_gate' the same with the tanh form of gelu."""
     ff: int
     act: str = "relu2"
     kind = "dense"
@@ -332,7 +399,7 @@ class HashedBigramSpec:
 
 @dataclass(frozen=True)
 class HybridLayerSpec:
-    mixer: object                       # Latent / Decay / Window / Conv attention spec | SsmSpec | PairedMixerSpec | RgLruSpec
+    mixer: object                       # Latent / Decay / Window / Conv attention spec | SsmSpec | PairedMixerSpec | RgLruSpec | RetentionSpec
     mlp: object = None                  # RoutedExpertsSpec | DenseMlpSpec | None: the layer has no feed-forward
 
 
@@ -368,6 +435,10 @@ class HybridSpec:
     bigram: HashedBigramSpec = None     # the embedding adds a hashed row of a second table chosen by the previous token
     # 'sandwich' blocks: a norm before AND after each sublayer (plain weights), x <- x + n1b(mixer(n1(x))), x <- x + n2b(ff(n2(x))).
     logit_scale: float = 1.0
+    # 'streams' blocks: `streams` copies of the residual; a sublayer reads u = sum_s in[s] x_s through an offset norm and its output y,
+    #              scaled per column, joins all of them at once, x_t <- sum_s mix[s, t] x_s + out[t] * y (learned per sublayer); the
+    #              embedding is normed, the model's end reads the sum of the streams.
+    streams: int = 1
     hybrid = True
 
     @property
@@ -597,6 +668,69 @@ def duparax_spec(cfg, name="duparax", tensor_shapes=None):
                       logit_scale=float(cfg.get("logit_scale", 1.0)))
 
 
+def _rotation_of(r, dim):
+    rot = RotarySpec(int(r["dims"]), float(r["base"]), halves=True)
+    if not 0 <= rot.dims <= dim or rot.dims % 2:
+        raise ValueError(f"rot.dims {rot.dims} (even) does not fit dim {dim}")
+    return rot
+
+
+def _grouped(m):
+    heads, kv_heads = int(m["heads"]), int(m["kv_heads"])
+    if kv_heads < 1 or heads % kv_heads:
+        raise ValueError(f"{heads} query heads do not divide into {kv_heads} key/value heads")
+    return heads, kv_heads
+
+
+def _sefuvik_mixer(kind, m, rank):
+    """rank(tensor) -> the inner size of a pair of low-rank matrices (the rows of the first one), asked for only where the mixer has them."""
+    plain = dict(qk_norm=False, distance_bias=False, talking_heads=False)
+    if kind == "attention":
+        heads, kv_heads = _grouped(m)
+        mask = m.get("mask") or {}
+        return WindowAttentionSpec(heads, kv_heads, int(m["dim"]), int(m["vdim"]), float(m["scale"]), window=int(mask.get("size") or 0), bias=True,
+                                   gate=False, keep_first=int(mask.get("keep_first") or 0), maps=2, diff=float(m["diff"]), **plain)
+    if kind == "retention":
+        decay = tuple(float(d) for d in m["decay"])
+        if len(decay) != m["heads"]:
+            raise ValueError(f"{len(decay)} decays for {m['heads']} heads")
+        return RetentionSpec(int(m["heads"]), int(m["dim"]), int(m["vdim"]), decay, _rotation_of(m["rot"], int(m["dim"])))
+    if kind == "parallel":
+        l, r = m["left"], m["right"]
+        heads, kv_heads = _grouped(l)
+        left = WindowAttentionSpec(heads, kv_heads, int(l["dim"]), int(l["vdim"]), float(l["scale"]), bias=False, gate=True,
+                                   rot=_rotation_of(l["rot"], int(l["dim"])), chunk=int((l.get("mask") or {}).get("size") or 0), sink=True, **plain)
+        heads, kv_heads = _grouped(r)
+        right = GatedDeltaSpec(heads, kv_heads, int(r["dim"]), int(r["vdim"]), int(r["conv"]), rank("a1"), rank("g1"))
+        return PairedMixerSpec(left, right, (float(m["left_scale"]), float(m["right_scale"])))
+    raise NotImplementedError(f"mixer type {kind!r}")
+
+
+def sefuvik_spec(cfg, name="sefuvik", tensor_shapes=None):
+    """config.json of a Sefuvik checkpoint -> HybridSpec.  Every size and constant is read from the config; the inner sizes of the
+    decay's and the gate's low-rank matrices are tensor shapes ('l<i>.mix.right.a1', '...g1': [rank, width])."""
+    layers = []
+    for i, entry in enumerate(cfg["layers"]):
+
+        def rank(tensor):
+            r = entry["mixer"]["right"]
+            if f"{tensor}_rank" in r:
+                return int(r[f"{tensor}_rank"])
+            if not tensor_shapes:
+                raise ValueError(f"layer {i}: the inner size of {tensor} is neither in the config nor a known tensor shape")
+            return int(tensor_shapes[f"l{i}.mix.right.{tensor}"][0])
+
+        mlp = entry.get("mlp")
+        if mlp is not None:
+            if mlp["kind"] != "dense":
+                raise NotImplementedError(f"feed-forward kind {mlp['kind']!r}")
+            mlp = DenseMlpSpec(int(mlp["ff"]), act="gelu_gate")
+        layers.append(HybridLayerSpec(_sefuvik_mixer(entry["type"], entry["mixer"], rank), mlp))
+    return HybridSpec(name=name, arch="sefuvik", width=int(cfg["width"]), vocab=int(cfg["vocab"]), layers=tuple(layers),
+                      norm_eps=float(cfg["norm"]["eps"]), norm_groups=1, conv_taps=1, embedding_scale=1.0,
+                      session_len=int(cfg.get("session_len", 0)), block="streams", tied_head=True, streams=int(cfg["streams"]))
+
+
 # config.json "architecture" -> spec builder, for checkpoints that are not HF `architectures` configs
 HYBRID_ARCHITECTURES = {"Gulozen": gulozen_spec, "Bodopel": bodopel_spec, "Lifuzen": lifuzen_spec, "Fogizen": fogizen_spec,
-                        "Duparax": duparax_spec}
+                        "Duparax": duparax_spec, "Sefuvik": sefuvik_spec}

@@ -102,9 +102,11 @@ class EmulatedHybridLib:
         ang = float(pos) * f
         c, s = (np.cos(ang) * a.rot.magnitude).astype(np.float32), (np.sin(ang) * a.rot.magnitude).astype(np.float32)
         out = v.copy()
-        u, w = v[..., 0:2 * a.rot.pairs:2], v[..., 1:2 * a.rot.pairs:2]
-        out[..., 0:2 * a.rot.pairs:2] = u * c - w * s
-        out[..., 1:2 * a.rot.pairs:2] = w * c + u * s
+        P = a.rot.pairs
+        one, two = (slice(0, P), slice(P, 2 * P)) if a.rot.halves else (slice(0, 2 * P, 2), slice(1, 2 * P, 2))
+        u, w = v[..., one], v[..., two]
+        out[..., one] = u * c - w * s
+        out[..., two] = w * c + u * s
         return out
 
     @staticmethod
@@ -265,7 +267,8 @@ class EmulatedHybridLib:
         base = int(ptrs[cu[seq] + pos // a.block_len]) + a.layer_off
         at = pos % a.block_len
         G, D, V = a.kv_heads, a.dim, a.vdim
-        return _f(base + 4 * at * G * D, G, D), _f(base + a.v_off + 4 * at * G * V, G, V)
+        GK = G * max(getattr(a, "maps", 1), 1)
+        return _f(base + 4 * at * GK * D, GK, D), _f(base + a.v_off + 4 * at * G * V, G, V)
 
     @staticmethod
     def _growth(a, pos):
@@ -277,10 +280,10 @@ class EmulatedHybridLib:
     def b200h_window_prep(self, args):
         a = args._obj
         assert a.dtype == F32
-        H, G, D, V = a.heads, a.kv_heads, a.dim, a.vdim
-        q, k, v = _rows(a.q, a.n, a.ld, H * D), _rows(a.k, a.n, a.ld, G * D), _rows(a.v, a.n, a.ld, G * V)
+        H, G, D, V, GV = a.heads * max(a.maps, 1), a.kv_heads * max(a.maps, 1), a.dim, a.vdim, a.kv_heads
+        q, k, v = _rows(a.q, a.n, a.ld, H * D), _rows(a.k, a.n, a.ld, G * D), _rows(a.v, a.n, a.ld, GV * V)
         if a.bias:
-            b = _f(a.bias, (H + G) * D + G * V)
+            b = _f(a.bias, (H + G) * D + GV * V)
             q, k, v = q + b[:H * D], k + b[H * D:(H + G) * D], v + b[(H + G) * D:]
         _f(a.qn, a.n, H * D)[:] = _unit(q, a.eps) * _f(a.q_norm, H * D) if a.q_norm else q
         kn = _unit(k, a.eps) * _f(a.k_norm, G * D) if a.k_norm else k
@@ -289,15 +292,15 @@ class EmulatedHybridLib:
         for t in range(a.n):
             kd, vd = self._kv(a, int(seqs[t]), int(poss[t]))
             kd[:] = kn[t].reshape(G, D)
-            vd[:] = v[t].reshape(G, V)
+            vd[:] = v[t].reshape(GV, V)
         return 0
 
     def b200h_window_attention(self, args):
         a = args._obj
-        H, G, D, V = a.heads, a.kv_heads, a.dim, a.vdim
+        H, G, D, V, M = a.heads, a.kv_heads, a.dim, a.vdim, max(a.maps, 1)
         rep = H // G
-        qn = _f(a.qn, a.n, H, D)
-        y = _f(a.y, a.n, H * V)
+        qn = _f(a.qn, a.n, H, M, D)
+        y = _rows(a.y, a.n, a.ld_y or H * V, H * V)
         gate = _rows(a.gate, a.n, a.ld_gate, H if a.gate_heads else H * V) if a.gate else None
         seqs, poss = _i(a.tok_seq, a.n), _i(a.tok_pos, a.n)
         for t in range(a.n):
@@ -305,13 +308,28 @@ class EmulatedHybridLib:
             lo = max(0, pos - a.window + 1) if a.window > 0 else 0
             if a.chunk > 0:
                 lo = max(lo, pos // a.chunk * a.chunk)
-            ks, vs = zip(*[self._kv(a, s, j) for j in range(lo, pos + 1)])
-            ks, vs = np.stack(ks), np.stack(vs)                                    # [L, G, D], [L, G, V]
-            dist = (pos - np.arange(lo, pos + 1)).astype(np.float32)
+            seen = np.array([j for j in range(pos + 1) if j >= lo or (a.window > 0 and j < a.keep_first)])
+            ks, vs = zip(*[self._kv(a, s, int(j)) for j in seen])
+            ks, vs = np.stack(ks).reshape(len(seen), G, M, D), np.stack(vs)        # [L, G, maps, D], [L, G, V]
+            if M == 2:
+                out = np.zeros((H, V), np.float32)
+                for h in range(H):
+                    both = []
+                    for b in range(2):
+                        e = (ks[:, h // rep, b] @ qn[t, h, b]) * np.float32(a.scale)
+                        e = np.exp(e - e.max())
+                        both.append(e / e.sum())
+                    out[h] = (both[0] - np.float32(a.lambda_) * both[1]) @ vs[:, h // rep]
+                if a.out_norm:
+                    out = _unit(out, a.eps)
+                y[t] = out.reshape(H * V) * np.float32(a.out_scale)
+                continue
+            ks = ks[:, :, 0]
+            dist = (pos - seen).astype(np.float32)
             wts = np.zeros((H, len(dist)), np.float32)
             raw = np.zeros((H, len(dist)), np.float32)
             for h in range(H):
-                sc = (ks[:, h // rep] @ qn[t, h]) * np.float32(a.scale)
+                sc = (ks[:, h // rep] @ qn[t, h, 0]) * np.float32(a.scale)
                 if a.softcap > 0:
                     sc = a.softcap * np.tanh(sc / a.softcap)
                 if a.r1:
@@ -333,7 +351,7 @@ class EmulatedHybridLib:
             out = np.stack([wts[h] @ vs[:, h // rep] for h in range(H)])
             if gate is not None:
                 out = out * (_sigmoid(gate[t])[:, None] if a.gate_heads else _sigmoid(gate[t]).reshape(H, V))
-            y[t] = out.reshape(H * V)
+            y[t] = out.reshape(H * V) * np.float32(a.out_scale)
         return 0
 
     def b200h_head_rope_prep(self, args, rot):
@@ -441,9 +459,14 @@ class EmulatedHybridLib:
         return 0
 
     def b200h_group_norm_gate(self, o, w, gate, ld_gate, n, count, groups, act, eps, y, dtype, stream):
+        return self.b200h_group_norm_gate_rows(o, w, gate, ld_gate, n, count, groups, act, eps, y, count, dtype, stream)
+
+    def b200h_group_norm_gate_rows(self, o, w, gate, ld_gate, n, count, groups, act, eps, y, ld_y, dtype, stream):
+        assert dtype == F32
         G = _rows(gate, n, ld_gate, count)
         g = G * _sigmoid(G) if act == 1 else _sigmoid(G)
-        _f(y, n, count)[:] = _unit(_f(o, n, groups, count // groups), eps).reshape(n, count) * _f(w, count) * g
+        wt = _f(w, count) if w else np.float32(1)
+        _rows(y, n, ld_y, count)[:] = _unit(_f(o, n, groups, count // groups), eps).reshape(n, count) * wt * g
         return 0
 
     def b200h_xielu(self, x, count, params, dtype, stream):
@@ -557,8 +580,127 @@ class EmulatedHybridLib:
         return 0
 
     def b200h_silu_mul_rows(self, gu, n, cols, out, dtype, stream):
+        return self.b200h_gate_mul_rows(gu, n, cols, 0, out, dtype, stream)
+
+    def b200h_gate_mul_rows(self, gu, n, cols, act, out, dtype, stream):
         G = _f(gu, n, 2, cols)
-        _f(out, n, cols)[:] = G[:, 0] * _sigmoid(G[:, 0]) * G[:, 1]
+        z = G[:, 0]
+        g = 0.5 * z * (1 + np.tanh(np.sqrt(2 / np.pi) * (z + 0.044715 * z ** 3))) if act else z * _sigmoid(z)
+        _f(out, n, cols)[:] = g * G[:, 1]
+        return 0
+
+    # ---- blocks of parallel residual streams, retention, gated delta rule
+    def b200h_embed_streams(self, tokens, table, scale, w_embed, x, streams, read, w_next, n, width, eps, h, dtype, stream):
+        assert dtype == F32
+        tok = _i(tokens, n)
+        e = _a(table, (int(tok.max()) + 1) * width).reshape(-1, width)[tok] * np.float32(scale)
+        if w_embed:
+            e = _unit(e, eps) * _f(w_embed, width)
+        X = _f(x, n, streams, width)
+        X[:] = e[:, None]
+        _f(h, n, width)[:] = _unit(np.einsum("s,nsw->nw", _a(read, streams), X), eps) * _f(w_next, width)
+        return 0
+
+    def b200h_join_streams(self, x, streams, y, ls, mix, out, read, w_next, rows, count, width, eps, write, u, h, dtype, stream):
+        assert dtype == F32
+        if count == 0:
+            return 0
+        at = _i(rows, count) if rows else np.arange(count)
+        X = _f(x, int(at.max()) + 1, streams, width)
+        v = X[at].copy()
+        if y:
+            Y = _f(y, int(at.max()) + 1, width)[at]
+            if ls:
+                Y = Y * _f(ls, width)
+            v = np.einsum("sd,nsw->ndw", _f(mix, streams, streams), v) + _a(out, streams)[None, :, None] * Y[:, None]
+            if write:
+                X[at] = v
+        total = np.einsum("s,nsw->nw", _a(read, streams), v) if read else v.sum(1)
+        if u:
+            _f(u, count, width)[:] = total
+        if h:
+            _f(h, count, width)[:] = _unit(total, eps) * _f(w_next, width)
+        return 0
+
+    def b200h_retention_prep(self, q, k, ld, n, heads, dim, k_scale, rot, tok_pos, qk, dtype, stream):
+        assert dtype == F32
+
+        class Holder:
+            pass
+        holder = Holder()
+        holder.rot = rot._obj
+        Q, K, pos = _rows(q, n, ld, heads * dim).reshape(n, heads, dim), _rows(k, n, ld, heads * dim).reshape(n, heads, dim), _i(tok_pos, n)
+        O = _f(qk, n, 2, heads, dim)
+        for t in range(n):
+            O[t, 0] = self._rot(Q[t], int(pos[t]), holder)
+            O[t, 1] = self._rot(K[t], int(pos[t]), holder) * np.float32(k_scale)
+        return 0
+
+    def b200h_retention_scan(self, qk, v, ld_v, decay, state, slot_stride, cu_q, seq_slot, batch, heads, dim, vdim, out, dtype, stream):
+        assert dtype == F32
+        cu, slots, lam = _i(cu_q, batch + 1), _i(seq_slot, batch), _a(decay, heads)
+        n = int(cu[batch])
+        QK, Vv, O = _f(qk, n, 2, heads, dim), _rows(v, n, ld_v, heads * vdim).reshape(n, heads, vdim), _f(out, n, heads, vdim)
+        for s in range(batch):
+            S = _f(int(state) + 4 * int(slots[s]) * slot_stride, heads, vdim, dim)            # [head][value][key]
+            for t in range(cu[s], cu[s + 1]):
+                for h in range(heads):
+                    S[h] = lam[h] * S[h] + np.outer(Vv[t, h], QK[t, 1, h])
+                    O[t, h] = S[h] @ QK[t, 0, h]
+        return 0
+
+    def b200h_low_rank_rate_decay(self, low, ld, a, bias, rate, n, heads, dim, rank, decay, dtype, stream):
+        assert dtype == F32
+        z = _rows(low, n, ld, rank) @ _f(a, rank, heads * dim) + _f(bias, heads * dim)
+        _f(decay, n, heads, dim)[:] = np.exp(-_a(rate, heads)[:, None] * np.logaddexp(0, z).reshape(n, heads, dim))
+        return 0
+
+    def b200h_delta_prep(self, args):
+        a = args._obj
+        assert a.dtype == F32
+        KD, HV = a.kv_heads * a.dim, a.heads * a.vdim
+        ch = 2 * KD + HV
+        cu, slots = _i(a.cu_q, a.batch + 1), _i(a.seq_slot, a.batch)
+        kept = {}                           # the state is advanced by the scan: put back what _conv_rows advances
+        for s in range(a.batch):
+            st = _f(int(a.conv_state) + 4 * int(slots[s]) * a.slot_stride, a.taps - 1, ch)
+            kept[s] = (st, st.copy())
+        y = self._conv_rows(_rows(a.u, a.n, a.ld, ch), _f(a.conv, a.taps, ch).T, None, a.conv_state, a.slot_stride, cu, slots, a.batch, a.taps)
+        for st, old in kept.values():
+            st[:] = old
+        y = y * _sigmoid(y)
+        qk = y[:, :2 * KD].reshape(a.n, 2, a.kv_heads, a.dim)
+        qk = qk / np.sqrt((qk * qk).sum(-1, keepdims=True) + np.float32(a.unit_eps))
+        qk[:, 0] *= np.float32(a.q_scale)
+        O = _f(a.qkv, a.n, ch)
+        O[:, :2 * KD], O[:, 2 * KD:] = qk.reshape(a.n, 2 * KD), y[:, 2 * KD:]
+        _f(a.kq, a.n, a.kv_heads)[:] = (qk[:, 0] * qk[:, 1]).sum(-1)
+        _f(a.beta, a.n, a.heads)[:] = _sigmoid(_rows(a.b, a.n, a.ld, a.heads))
+        return 0
+
+    def b200h_delta_scan(self, args):
+        a = args._obj
+        assert a.dtype == F32
+        KD, HV = a.kv_heads * a.dim, a.heads * a.vdim
+        ch = 2 * KD + HV
+        QKV, G, beta, O = _f(a.qkv, a.n, ch), _f(a.decay, a.n, a.heads, a.dim), _f(a.beta, a.n, a.heads), _f(a.out, a.n, a.heads, a.vdim)
+        U, cu, slots = _rows(a.u, a.n, a.ld, ch), _i(a.cu_q, a.batch + 1), _i(a.seq_slot, a.batch)
+        for s in range(a.batch):
+            lo, hi = cu[s], cu[s + 1]
+            if lo == hi:
+                continue
+            S = _f(int(a.state) + 4 * int(slots[s]) * a.slot_stride, a.heads, a.vdim, a.dim)  # [head][value][key]
+            for t in range(lo, hi):
+                for h in range(a.heads):
+                    kh = h // (a.heads // a.kv_heads)
+                    q, k = QKV[t, kh * a.dim:(kh + 1) * a.dim], QKV[t, KD + kh * a.dim:KD + (kh + 1) * a.dim]
+                    v = QKV[t, 2 * KD + h * a.vdim:2 * KD + (h + 1) * a.vdim]
+                    S[h] *= G[t, h]
+                    S[h] += np.outer(beta[t, h] * (v - S[h] @ k), k)
+                    O[t, h] = S[h] @ q
+            st = _f(int(a.conv_state) + 4 * int(slots[s]) * a.slot_stride, a.taps - 1, ch)
+            full = np.concatenate([st, U[lo:hi]], 0)
+            st[:] = full[full.shape[0] - (a.taps - 1):]
         return 0
 
     # ---- parallel blocks, convolved rotary attention, state-space mixer
