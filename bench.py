@@ -129,6 +129,26 @@ def duparax_bench_config(z):
                         "mlp": dense if i == 0 else moe} for i, t in enumerate(HYBRID_LAYERS)]}
 
 
+def sefuvik_bench_config(z, window=1024, chunk=2048):
+    """A Sefuvik config.json (dict) of size `z`: four residual streams; differential attention with the dense decoder's head count and value
+    width (two maps of 64 dimensions per head, a window of 1024 keys that keeps the first 4), then two parallel layers around a retention
+    layer -- chunked attention with the dense decoder's head geometry (64 of 128 dimensions turn, chunks of 2048 keys: the bench's contexts
+    stay inside the first chunk) beside width / 64 heads of a 64 x 64 gated delta rule (4 taps, low-rank matrices of inner size 64);
+    width / 128 retention heads of 128 x 128 --, each with a gated feed-forward of the dense decoder's size."""
+    d = z["dense"]
+    att = {"heads": d["heads"], "kv_heads": d["kv_heads"], "dim": 64, "vdim": 128, "mask": {"size": window, "keep_first": 4}, "scale": 0.125, "diff": 0.4}
+    left = {"heads": d["heads"], "kv_heads": d["kv_heads"], "dim": 128, "vdim": 128, "mask": {"size": chunk}, "scale": 128 ** -0.5,
+            "rot": {"dims": 64, "base": 10000.0}}
+    n = z["width"] // 64
+    right = {"heads": n, "kv_heads": n, "dim": 64, "vdim": 64, "conv": 4, "a1_rank": 64, "g1_rank": 64}
+    n = z["width"] // 128
+    ret = {"heads": n, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** -(5 + 5 * h / n) for h in range(n)], "rot": {"dims": 128, "base": 10000.0}}
+    pair = {"left": left, "right": right, "left_scale": 0.8, "right_scale": 1.1}
+    return {"architecture": "Sefuvik", "norm": {"eps": 1e-6}, "vocab": HYBRID_VOCAB, "width": z["width"], "streams": 4,
+            "layers": [{"type": t, "mixer": m, "mlp": {"kind": "dense", "ff": d["inter"]}}
+                       for t, m in (("attention", att), ("parallel", pair), ("retention", ret), ("parallel", pair))]}
+
+
 def _hybrid_leg(torch, spec, batch, ctx, steps, warm, session, blocks):
     """One hybrid decoder through its engine: throughput, then per-operator device time (eight more decode steps, then one fresh
     4096-row prefill step, bracketed by CUDA events)."""
@@ -195,7 +215,7 @@ def run_hybrid(args):
     from lmdeploy_b200.messages import TurbomindEngineConfig
     from lmdeploy_b200.turbomind import ModelSpec
     from lmdeploy_b200.turbomind.engine import TurboMind
-    from lmdeploy_b200.turbomind.specs import bodopel_spec, duparax_spec, fogizen_spec, gulozen_spec, lifuzen_spec
+    from lmdeploy_b200.turbomind.specs import bodopel_spec, duparax_spec, fogizen_spec, gulozen_spec, lifuzen_spec, sefuvik_spec
     z = HYBRID_SIZES[args.hybrid]
     batch, ctx, steps, warm = args.hybrid_batch, args.hybrid_ctx, args.steps, max(args.warmup, 3)
     session = 2 * ctx + warm + steps + 16
@@ -212,6 +232,8 @@ def run_hybrid(args):
             spec = fogizen_spec(fogizen_bench_config(z), name=f"fogizen-{args.hybrid}")
         elif args.hybrid_design == "duparax":
             spec = duparax_spec(duparax_bench_config(z), name=f"duparax-{args.hybrid}")
+        elif args.hybrid_design == "sefuvik":
+            spec = sefuvik_spec(sefuvik_bench_config(z), name=f"sefuvik-{args.hybrid}")
         else:
             spec = gulozen_spec(hybrid_config(z), name=f"gulozen-{args.hybrid}")
         out["hybrid"] = _hybrid_leg(torch, spec, batch, ctx, steps, warm, session, blocks)
@@ -227,6 +249,10 @@ def run_hybrid(args):
             # the closest existing model -- paired mixers of attention and a channel-decay recurrence, dense and routed gated feed-forwards
             out["closest"] = dict(_hybrid_leg(torch, fogizen_spec(fogizen_bench_config(z), name=f"fogizen-{args.hybrid}"), batch, ctx, steps,
                                               warm, session, blocks), design="fogizen")
+        if args.hybrid_design == "sefuvik":
+            # the closest existing model -- attention beside a linear recurrence with a decay per key channel, gated feed-forwards
+            out["closest"] = dict(_hybrid_leg(torch, duparax_spec(duparax_bench_config(z), name=f"duparax-{args.hybrid}"), batch, ctx, steps,
+                                              warm, session, blocks), design="duparax")
         d = z["dense"]
         dspec = ModelSpec(f"dense-{args.hybrid}", "llama", d["hidden"], len(HYBRID_LAYERS), d["heads"], d["kv_heads"], d["inter"], HYBRID_VOCAB,
                           1e4, weight_format="fp16")
@@ -261,14 +287,15 @@ def parse():
     ap.add_argument("--hybrid", default=None, choices=list(HYBRID_SIZES),
                     help="instead of the default workload: prefill and decode tokens/s of a hybrid decoder of this size (--hybrid-design) "
                          "beside the dense decoder of equal size, both through the engine (random weights)")
-    ap.add_argument("--hybrid-design", default="gulozen", choices=["gulozen", "bodopel", "lifuzen", "fogizen", "duparax"],
+    ap.add_argument("--hybrid-design", default="gulozen", choices=["gulozen", "bodopel", "lifuzen", "fogizen", "duparax", "sefuvik"],
                     help="which hybrid design --hybrid builds: Gulozen (latent / decayed linear attention, routed experts), Bodopel "
                          "(windowed attention with grouped key/value heads, dense feed-forward) or Lifuzen (parallel blocks: convolved rotary "
                          "attention with a sink / state-space mixer, sigmoid-routed squared-relu experts; also runs Gulozen of equal size, the "
                          "closest existing model, beside it) or Fogizen (shared-norm blocks with token shift: chunked rotary attention beside a "
                          "channel-decay recurrence in every layer, dense and group-routed experts; also runs Lifuzen of equal size beside it) or Duparax (norms on both ends of "
                          "every sublayer: attention beside gated linear attention / RG-LRU, dense and routed feed-forwards with a shared expert; "
-                         "also runs Fogizen of equal size beside it)")
+                         "also runs Fogizen of equal size beside it) or Sefuvik (parallel residual streams: differential attention / retention / "
+                         "chunked attention beside the gated delta rule, gated feed-forwards; also runs Duparax of equal size beside it)")
     ap.add_argument("--hybrid-batch", type=int, default=32)
     ap.add_argument("--hybrid-ctx", type=int, default=1024)
     ap.add_argument("--no-graph", action="store_true", help="do not capture the step in a CUDA graph")

@@ -5,6 +5,35 @@
 // Number formats: projections (T) are read once; rotated queries and keys, the convolutions' outputs, unit vectors, decays, step sizes,
 // the recurrence and its state are float.
 
+// z / (1 + exp(-z)) by the hardware's approximate exponential and division (relative error about 1e-6)
+__device__ __forceinline__ float silu_fast(float z) { return __fdividef(z, 1.0f + __expf(-z)); }
+
+// Two floats of one 64-bit register pair: a * b and a * b + c by sm_100's packed instructions
+__device__ __forceinline__ unsigned long long pack2(float lo, float hi)
+{
+    unsigned long long r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
+    return r;
+}
+__device__ __forceinline__ float sum2(unsigned long long v)
+{
+    float lo, hi;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v));
+    return lo + hi;
+}
+__device__ __forceinline__ unsigned long long mul2(unsigned long long a, unsigned long long b)
+{
+    unsigned long long r;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+    return r;
+}
+__device__ __forceinline__ unsigned long long fma2(unsigned long long a, unsigned long long b, unsigned long long c)
+{
+    unsigned long long r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+    return r;
+}
+
 // One block per row: every head of q and k turns by the row's position (first 2 * rot.pairs dimensions), k is multiplied by k_scale.
 // qk: float [n, 2 * heads * dim] = rotated q | rotated k.  Shared memory: 2 * rot.pairs floats of cos / sin.
 template <typename T>
@@ -57,7 +86,8 @@ struct DeltaPrep {
 };
 
 // A thread's V channels c .. c + V - 1 of ROWS consecutive rows from t0: silu(sum_j w[j, c] u[t - taps + 1 + j, c]).  Rows before the
-// step's first row of a sequence come from its state.  TAPS >= taps: the leading weights are zero.
+// step's first row of a sequence come from its state.  TAPS >= taps: the leading weights are zero.  The rows' loads and those of the
+// rows before t0 are issued before the sequence is known; what belongs to another sequence is replaced by the state afterwards.
 template <typename T, int TAPS, int ROWS, int V>
 __device__ __forceinline__ void conv_silu_rows(const T* __restrict__ u, int64_t ld, const DeltaPrep& d, int channels, int c, int t0, int rows,
                                                float (&y)[ROWS][V])
@@ -67,32 +97,38 @@ __device__ __forceinline__ void conv_silu_rows(const T* __restrict__ u, int64_t 
     for (int r = 0; r < ROWS; ++r)
         if (r < rows) load_vals<V>(u + (size_t)(t0 + r) * ld + c, x[r]);
 #pragma unroll
+    for (int j = 0; j < TAPS - 1; ++j) {
+        const int src = t0 - (TAPS - 1) + j;
+        if (j >= TAPS - d.taps && src >= 0) load_vals<V>(u + (size_t)src * ld + c, win[j]);
+        else
+#pragma unroll
+            for (int e = 0; e < V; ++e) win[j][e] = 0.f;
+    }
+#pragma unroll
     for (int j = 0; j < TAPS; ++j) {
         if (j >= TAPS - d.taps) load_vals<V>(d.w + (size_t)(j - (TAPS - d.taps)) * channels + c, wt[j]);
         else
 #pragma unroll
             for (int e = 0; e < V; ++e) wt[j][e] = 0.f;
     }
-    int seq = -1;
+    int s = d.tok_seq[t0], first = d.cu_q[s], end = d.cu_q[s + 1];
 #pragma unroll
     for (int r = 0; r < ROWS; ++r) {
         if (r < rows) {
-            const int s = d.tok_seq[t0 + r];
-            if (s != seq) {                                   // this block's first row of the sequence: its predecessors from the step or the state
-                seq = s;
-                const int first = d.cu_q[s], local = t0 + r - first;
+            if (t0 + r >= end) {                              // the next sequence that has rows in this step starts here
+                s = d.tok_seq[t0 + r];
+                first = t0 + r;
+                end = d.cu_q[s + 1];
+            }
+            const int local = t0 + r - first;
+            if (local < d.taps - 1 && (r == 0 || local == 0)) {
                 const float* st = d.state + (int64_t)d.seq_slot[s] * d.slot_stride;
 #pragma unroll
                 for (int j = 0; j < TAPS - 1; ++j) {
                     const int src = local - (TAPS - 1) + j;
+                    if (j >= TAPS - d.taps && src < 0)
 #pragma unroll
-                    for (int e = 0; e < V; ++e) win[j][e] = 0.f;
-                    if (j >= TAPS - d.taps) {
-                        if (src >= 0) load_vals<V>(u + (size_t)(first + src) * ld + c, win[j]);
-                        else
-#pragma unroll
-                            for (int e = 0; e < V; ++e) win[j][e] = st[(size_t)(src + d.taps - 1) * channels + c + e];
-                    }
+                        for (int e = 0; e < V; ++e) win[j][e] = st[(size_t)(src + d.taps - 1) * channels + c + e];
                 }
             }
 #pragma unroll
@@ -101,7 +137,7 @@ __device__ __forceinline__ void conv_silu_rows(const T* __restrict__ u, int64_t 
                 float acc = 0.f;
 #pragma unroll
                 for (int j = 0; j < TAPS; ++j) acc = fmaf(wt[j][e], win[j][e], acc);
-                y[r][e] = silu_f(acc);
+                y[r][e] = silu_fast(acc);
 #pragma unroll
                 for (int j = 0; j < TAPS - 1; ++j) win[j][e] = win[j + 1][e];
             }
@@ -111,17 +147,19 @@ __device__ __forceinline__ void conv_silu_rows(const T* __restrict__ u, int64_t 
 
 // What the gated delta rule reads, from the projection's columns u = q | k | v and b (one column per head):  every channel's convolution
 // and silu; q and k of every head divided by sqrt(sum of squares + unit_eps), q times q_scale; their dot product; beta = sigmoid(b).
-// grid (row groups, kv_heads + blocks of v channels), 128 threads: block y < kv_heads takes query head y and key head y (through shared
-// memory [ROWS][2 * dim]), the others V * 128 channels of v each; block y == 0 also the row group's betas.
+// grid (row groups, blocks of key heads + blocks of v channels), 128 threads: the first `head_blocks` blocks take `per` query heads and the
+// same key heads each (through shared memory [ROWS][per][2 * dim]), the others V * 128 channels of v; block y == 0 also the row group's
+// betas.
 template <typename T, int TAPS, int ROWS, int V>
-__global__ void __launch_bounds__(128) delta_prep_kernel(const T* __restrict__ u, const T* __restrict__ b, int64_t ld, DeltaPrep d)
+__global__ void __launch_bounds__(128, ROWS == 8 ? 6 : 1) delta_prep_kernel(const T* __restrict__ u, const T* __restrict__ b, int64_t ld, DeltaPrep d, int per,
+                                                        int head_blocks)
 {
     extern __shared__ __align__(16) float dp_smem[];
-    const int t0 = blockIdx.x * ROWS, rows = min(ROWS, d.n - t0), g = blockIdx.y, D = d.dim, KD = d.kv_heads * D;
+    const int t0 = blockIdx.x * ROWS, rows = min(ROWS, d.n - t0), D = d.dim, KD = d.kv_heads * D;
     const int channels = 2 * KD + d.heads * d.vdim;
     float y[ROWS][V];
-    if (g >= d.kv_heads) {
-        const int c = 2 * KD + ((g - d.kv_heads) * 128 + threadIdx.x) * V;
+    if ((int)blockIdx.y >= head_blocks) {
+        const int c = 2 * KD + ((blockIdx.y - head_blocks) * 128 + threadIdx.x) * V;
         if (c >= channels) return;
         conv_silu_rows<T, TAPS, ROWS, V>(u, ld, d, channels, c, t0, rows, y);
 #pragma unroll
@@ -129,24 +167,25 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(const T* __restrict__ u
             if (r < rows) store_vals<V>(d.qkv + (size_t)(t0 + r) * channels + c, y[r]);
         return;
     }
-    for (int i = threadIdx.x * V; i < 2 * D; i += 128 * V) {
-        const int c = i < D ? g * D + i : KD + g * D + i - D;
-        conv_silu_rows<T, TAPS, ROWS, V>(u, ld, d, channels, c, t0, rows, y);
+    const int g0 = blockIdx.y * per, heads = min(per, d.kv_heads - g0), span = heads * D;      // q channels g0 D .. + span, k the same
+    for (int i = threadIdx.x * V; i < 2 * span; i += 128 * V) {
+        const int key = i >= span, at = key ? i - span : i, g = at / D;
+        conv_silu_rows<T, TAPS, ROWS, V>(u, ld, d, channels, key * KD + g0 * D + at, t0, rows, y);
+        float* dst = dp_smem + g * 2 * D + key * D + at - g * D;
 #pragma unroll
         for (int r = 0; r < ROWS; ++r)
-            if (r < rows)
-#pragma unroll
-                for (int e = 0; e < V; ++e) dp_smem[r * 2 * D + i + e] = y[r][e];
+            if (r < rows) store_vals<V>(dst + (size_t)r * per * 2 * D, y[r]);
     }
-    if (g == 0)
+    if (blockIdx.y == 0)
         for (int i = threadIdx.x; i < rows * d.heads; i += 128) {
             const int r = i / d.heads, h = i - r * d.heads;
             d.beta[(size_t)(t0 + r) * d.heads + h] = sigmoid_f(to_f(b[(size_t)(t0 + r) * ld + h]));
         }
     __syncthreads();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    for (int r = warp; r < rows; r += 4) {
-        const float* q = dp_smem + r * 2 * D;
+    for (int it = warp; it < rows * heads; it += 4) {
+        const int r = it / heads, g = it - r * heads;
+        const float* q = dp_smem + (size_t)(r * per + g) * 2 * D;
         const float* k = q + D;
         float sq = 0.f, sk = 0.f, qk = 0.f;
         for (int i = lane; i < D; i += 32) {
@@ -158,12 +197,17 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(const T* __restrict__ u
         sk = warp_sum(sk);
         qk = warp_sum(qk);
         const float rq = d.q_scale / sqrtf(sq + d.unit_eps), rk = 1.0f / sqrtf(sk + d.unit_eps);
-        float* out = d.qkv + (size_t)(t0 + r) * channels + g * D;
-        for (int i = lane; i < D; i += 32) {
-            out[i] = q[i] * rq;
-            out[KD + i] = k[i] * rk;
+        float* out = d.qkv + (size_t)(t0 + r) * channels + (size_t)(g0 + g) * D;
+        for (int i = lane * V; i < D; i += 32 * V) {
+            float a[V], c[V];
+            load_vals<V>(q + i, a);
+            load_vals<V>(k + i, c);
+#pragma unroll
+            for (int e = 0; e < V; ++e) { a[e] *= rq; c[e] *= rk; }
+            store_vals<V>(out + i, a);
+            store_vals<V>(out + KD + i, c);
         }
-        if (lane == 0) d.kq[(size_t)(t0 + r) * d.kv_heads + g] = qk * rq * rk;
+        if (lane == 0) d.kq[(size_t)(t0 + r) * d.kv_heads + g0 + g] = qk * rq * rk;
     }
 }
 
@@ -196,13 +240,40 @@ __device__ __forceinline__ void copy_async16(float* dst, const float* src)
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((unsigned)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
 }
 
+// Where the values come from: the projection (T, retention) or the convolution (float, delta)
+template <typename T, bool DELTA> struct HeadScanValue {
+    typedef T type;
+    static __device__ __forceinline__ const T* pick(const T* t, const float*) { return t; }
+};
+template <typename T> struct HeadScanValue<T, true> {
+    typedef float type;
+    static __device__ __forceinline__ const float* pick(const T*, const float* f) { return f; }
+};
+
+// part[r] of eight neighbouring lanes -> the sum over the lanes of part[p] at lane p
+__device__ __forceinline__ float scatter_sum8(float (&part)[8], int p)
+{
+#pragma unroll
+    for (int m = 4; m > 0; m >>= 1) {
+        const bool upper = p & m;
+#pragma unroll
+        for (int i = 0; i < m; ++i) {
+            const float give = upper ? part[i] : part[i + m], keep = upper ? part[i + m] : part[i];
+            part[i] = keep + __shfl_xor_sync(0xffffffffu, give, m);
+        }
+    }
+    return part[0];
+}
+
 // Per head, S a [dim, vdim] float matrix per sequence, columns independent:
 //   retention:  S <- decay_h S + k v^T;  o = S^T q
 //   delta:      S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q = (diag(g) S_old)^T q + u (k . q)
-// The delta form takes both dot products of the decayed state in ONE pass and one round of shuffles; k . q comes from the preparation.
+// The delta form takes both dot products of the decayed state in ONE pass; k . q comes from the preparation.
 // Eight lanes own a value column: lane p keeps the state's entries 4 p + 32 e .. 4 p + 32 e + 3 in registers (e < NE) for NC columns, so a
-// warp holds 4 NC columns and a row costs three shuffles per sum and no block barrier.  R rows of q, k and decays pass through shared
-// memory at a time (asynchronous copies, double-buffered), v through registers (lane p of a column's eight holds row p's value).
+// warp holds 4 NC columns and rows meet no block barrier.  R = 8 rows of q, k and decays pass through shared memory at a time
+// (asynchronous copies, double-buffered), v through registers (lane p of a column's eight holds row p's value).  S^T k is summed over
+// the eight lanes row by row (the next row needs it); the R rows' partial S^T q are kept and summed together, seven shuffles that leave
+// row p's sum with lane p, which stores it.
 // blockDim (32, 4); grid (heads * ceil(vdim / (16 NC)), batch).  Entries past dim hold zeros and stay zero.
 template <typename T, bool DELTA, int NE, int NC>
 __global__ void __launch_bounds__(128) head_scan_kernel(HeadScan g, const T* __restrict__ v_t, const float* __restrict__ v_f)
@@ -216,64 +287,93 @@ __global__ void __launch_bounds__(128) head_scan_kernel(HeadScan g, const T* __r
     const int col = (blockIdx.x - h * groups) * 16 * NC + w * 4 * NC + (lane >> 3) * NC;
     float* sp = g.state + (int64_t)g.seq_slot[s] * g.slot_stride + (size_t)h * g.vdim * D;
     const bool vec = D % 4 == 0 && (reinterpret_cast<uintptr_t>(sp) & 15) == 0;
-    float S[NC][NE * 4];
+    unsigned long long S[NC][NE * 2];                         // pairs of neighbouring entries
 #pragma unroll
     for (int c = 0; c < NC; ++c)
 #pragma unroll
         for (int e = 0; e < NE; ++e) {
+            S[c][2 * e] = S[c][2 * e + 1] = 0ull;
             const int d = 4 * p + 32 * e;
-            const float* src = sp + (size_t)(col + c) * D + d;
-            if (vec && col + c < g.vdim && d < D) {
-                const float4 q4 = *reinterpret_cast<const float4*>(src);
-                S[c][4 * e] = q4.x; S[c][4 * e + 1] = q4.y; S[c][4 * e + 2] = q4.z; S[c][4 * e + 3] = q4.w;
-            } else {
-#pragma unroll
-                for (int i = 0; i < 4; ++i) S[c][4 * e + i] = (col + c < g.vdim && d + i < D) ? src[i] : 0.f;
+            if (vec && col + c < g.vdim && d < D) {           // all of a thread's reads are in flight together
+                const ulonglong2 q4 = *reinterpret_cast<const ulonglong2*>(sp + (size_t)(col + c) * D + d);
+                S[c][2 * e] = q4.x;
+                S[c][2 * e + 1] = q4.y;
             }
         }
+    if (!vec) {
+#pragma unroll
+        for (int c = 0; c < NC; ++c)
+#pragma unroll
+            for (int e = 0; e < 2 * NE; ++e) {
+                const int d = 4 * p + 32 * (e / 2) + 2 * (e & 1);
+                const float* src = sp + (size_t)(col + c) * D + d;
+                const bool live = col + c < g.vdim;
+                S[c][e] = pack2(live && d < D ? src[0] : 0.f, live && d + 1 < D ? src[1] : 0.f);
+            }
+    }
     for (int i = tid; i < 2 * STAGE; i += 128) hs_smem[i] = 0.f;
     __syncthreads();
-    const float lam = DELTA ? 0.f : g.decay[h];
+    const unsigned long long lam = DELTA ? 0ull : pack2(g.decay[h], g.decay[h]);
     const size_t hd = (size_t)g.heads * D;
+    // this thread's 16-byte pieces of a stage: row and first column
+    constexpr int PIECES = (R * NE * 8 + 127) / 128;
+    int pr[PIECES], pc[PIECES];
+#pragma unroll
+    for (int i = 0; i < PIECES; ++i) {
+        pr[i] = (tid + i * 128) / (D / 4 > 0 ? D / 4 : 1);
+        pc[i] = 4 * (tid + i * 128 - pr[i] * (D / 4));
+    }
+    const float* q_at = g.q + (size_t)kh * D;
+    const float* k_at = g.k + (size_t)kh * D;
+    const float* d_at = DELTA ? g.decay + (size_t)h * D : nullptr;
     // rows [t0, t0 + R) into stage buffer b
     auto stage_rows = [&](int t0, int b) {
         float* buf = hs_smem + b * STAGE;
-        const int rows = min(R, last - t0), per = g.aligned ? D / 4 : D;
-        for (int i = tid; i < rows * per; i += 128) {
-            const int r = i / per, c = i - r * per;
-            const size_t t = (size_t)(t0 + r);
-            if (g.aligned) {
-                copy_async16(buf + r * DP + 4 * c, g.q + t * g.ld_qk + (size_t)kh * D + 4 * c);
-                copy_async16(buf + (R + r) * DP + 4 * c, g.k + t * g.ld_qk + (size_t)kh * D + 4 * c);
-                if (DELTA) copy_async16(buf + (2 * R + r) * DP + 4 * c, g.decay + t * hd + (size_t)h * D + 4 * c);
-            } else {
-                copy_async4(buf + r * DP + c, g.q + t * g.ld_qk + (size_t)kh * D + c);
-                copy_async4(buf + (R + r) * DP + c, g.k + t * g.ld_qk + (size_t)kh * D + c);
-                if (DELTA) copy_async4(buf + (2 * R + r) * DP + c, g.decay + t * hd + (size_t)h * D + c);
+        const int rows = min(R, last - t0);
+        if (g.aligned) {
+#pragma unroll
+            for (int i = 0; i < PIECES; ++i) {
+                if (pr[i] < rows) {
+                    const size_t t = (size_t)(t0 + pr[i]);
+                    float* dst = buf + pr[i] * DP + pc[i];
+                    copy_async16(dst, q_at + t * g.ld_qk + pc[i]);
+                    copy_async16(dst + R * DP, k_at + t * g.ld_qk + pc[i]);
+                    if (DELTA) copy_async16(dst + 2 * R * DP, d_at + t * hd + pc[i]);
+                }
+            }
+        } else {
+            for (int i = tid; i < rows * D; i += 128) {
+                const int r = i / D, c = i - r * D;
+                const size_t t = (size_t)(t0 + r);
+                copy_async4(buf + r * DP + c, q_at + t * g.ld_qk + c);
+                copy_async4(buf + (R + r) * DP + c, k_at + t * g.ld_qk + c);
+                if (DELTA) copy_async4(buf + (2 * R + r) * DP + c, d_at + t * hd + c);
             }
         }
         if (DELTA && tid < 2 * rows) {
             const int r = tid >> 1;
-            if (tid & 1) copy_async4(buf + 3 * R * DP + R + r, g.kq + (size_t)(t0 + r) * g.kv_heads + kh);
-            else copy_async4(buf + 3 * R * DP + r, g.beta + (size_t)(t0 + r) * g.heads + h);
+            if (tid & 1) copy_async4(buf + 3 * R * DP + tid, g.kq + (size_t)(t0 + r) * g.kv_heads + kh);
+            else copy_async4(buf + 3 * R * DP + tid, g.beta + (size_t)(t0 + r) * g.heads + h);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
-    float vn[NC];
+    typedef typename HeadScanValue<T, DELTA>::type TV;
+    const TV* v = HeadScanValue<T, DELTA>::pick(v_t, v_f);
+    TV vn[NC];                                                // as stored: a conversion here would wait for the load
     auto load_v = [&](int t0) {
 #pragma unroll
         for (int c = 0; c < NC; ++c) {
             const size_t at = (size_t)(t0 + p) * g.ld_v + (size_t)h * g.vdim + col + c;
-            vn[c] = (t0 + p < last && col + c < g.vdim) ? (DELTA ? v_f[at] : to_f(v_t[at])) : 0.f;
+            vn[c] = (t0 + p < last && col + c < g.vdim) ? v[at] : from_f<TV>(0.f);
         }
     };
     stage_rows(first, 0);
     load_v(first);
     int b = 0;
     for (int t0 = first; t0 < last; t0 += R, b ^= 1) {
-        float vc[NC], oc[NC];
+        float vc[NC], oc[NC], part[NC][R];
 #pragma unroll
-        for (int c = 0; c < NC; ++c) { vc[c] = vn[c]; oc[c] = 0.f; }
+        for (int c = 0; c < NC; ++c) { vc[c] = to_f(vn[c]); oc[c] = 0.f; }
         if (t0 + R < last) {
             stage_rows(t0 + R, b ^ 1);                       // in flight while the staged rows are computed
             load_v(t0 + R);
@@ -283,64 +383,74 @@ __global__ void __launch_bounds__(128) head_scan_kernel(HeadScan g, const T* __r
         }
         __syncthreads();
         const float* buf = hs_smem + b * STAGE + 4 * p;
+        const float* row_nums = hs_smem + b * STAGE + 3 * R * DP;         // delta: (beta, k . q) of every row
         const int rows = min(R, last - t0);
-#pragma unroll 2
-        for (int r = 0; r < rows; ++r) {
-            float4 k4[NE];
-            float a[NC][2], o[NC][2], vr[NC];
+        auto row = [&](int r) {
+            unsigned long long k2[NE * 2], a[NC][2], o[NC][2];
+            float vr[NC];
 #pragma unroll
             for (int c = 0; c < NC; ++c) {
-                a[c][0] = a[c][1] = o[c][0] = o[c][1] = 0.f;
+                a[c][0] = a[c][1] = o[c][0] = o[c][1] = 0ull;
                 vr[c] = __shfl_sync(0xffffffffu, vc[c], (lane & 24) | r);
             }
 #pragma unroll
             for (int e = 0; e < NE; ++e) {
-                const float4 q4 = *reinterpret_cast<const float4*>(buf + r * DP + 32 * e);
-                k4[e] = *reinterpret_cast<const float4*>(buf + (R + r) * DP + 32 * e);
+                const ulonglong2 q4 = *reinterpret_cast<const ulonglong2*>(buf + r * DP + 32 * e);
+                const ulonglong2 k4 = *reinterpret_cast<const ulonglong2*>(buf + (R + r) * DP + 32 * e);
+                k2[2 * e] = k4.x;
+                k2[2 * e + 1] = k4.y;
                 if (DELTA) {
-                    const float4 g4 = *reinterpret_cast<const float4*>(buf + (2 * R + r) * DP + 32 * e);
+                    const ulonglong2 g4 = *reinterpret_cast<const ulonglong2*>(buf + (2 * R + r) * DP + 32 * e);
 #pragma unroll
                     for (int c = 0; c < NC; ++c) {
-                        float* st = S[c] + 4 * e;
-                        st[0] *= g4.x; st[1] *= g4.y; st[2] *= g4.z; st[3] *= g4.w;
-                        a[c][0] = fmaf(st[0], k4[e].x, a[c][0]); o[c][0] = fmaf(st[0], q4.x, o[c][0]);
-                        a[c][1] = fmaf(st[1], k4[e].y, a[c][1]); o[c][1] = fmaf(st[1], q4.y, o[c][1]);
-                        a[c][0] = fmaf(st[2], k4[e].z, a[c][0]); o[c][0] = fmaf(st[2], q4.z, o[c][0]);
-                        a[c][1] = fmaf(st[3], k4[e].w, a[c][1]); o[c][1] = fmaf(st[3], q4.w, o[c][1]);
+                        S[c][2 * e] = mul2(S[c][2 * e], g4.x);
+                        S[c][2 * e + 1] = mul2(S[c][2 * e + 1], g4.y);
+                        a[c][0] = fma2(S[c][2 * e], k4.x, a[c][0]);
+                        a[c][1] = fma2(S[c][2 * e + 1], k4.y, a[c][1]);
+                        o[c][0] = fma2(S[c][2 * e], q4.x, o[c][0]);
+                        o[c][1] = fma2(S[c][2 * e + 1], q4.y, o[c][1]);
                     }
                 } else {
 #pragma unroll
                     for (int c = 0; c < NC; ++c) {
-                        float* st = S[c] + 4 * e;
-                        st[0] = fmaf(lam, st[0], k4[e].x * vr[c]); o[c][0] = fmaf(st[0], q4.x, o[c][0]);
-                        st[1] = fmaf(lam, st[1], k4[e].y * vr[c]); o[c][1] = fmaf(st[1], q4.y, o[c][1]);
-                        st[2] = fmaf(lam, st[2], k4[e].z * vr[c]); o[c][0] = fmaf(st[2], q4.z, o[c][0]);
-                        st[3] = fmaf(lam, st[3], k4[e].w * vr[c]); o[c][1] = fmaf(st[3], q4.w, o[c][1]);
+                        const unsigned long long v2 = pack2(vr[c], vr[c]);
+                        S[c][2 * e] = fma2(lam, S[c][2 * e], mul2(k4.x, v2));
+                        S[c][2 * e + 1] = fma2(lam, S[c][2 * e + 1], mul2(k4.y, v2));
+                        o[c][0] = fma2(S[c][2 * e], q4.x, o[c][0]);
+                        o[c][1] = fma2(S[c][2 * e + 1], q4.y, o[c][1]);
                     }
                 }
             }
-            const float beta = DELTA ? hs_smem[b * STAGE + 3 * R * DP + r] : 0.f, kq = DELTA ? hs_smem[b * STAGE + 3 * R * DP + R + r] : 0.f;
+            const float2 nums = DELTA ? *reinterpret_cast<const float2*>(row_nums + 2 * r) : make_float2(0.f, 0.f);
 #pragma unroll
             for (int c = 0; c < NC; ++c) {
-                float oo = o[c][0] + o[c][1], aa = a[c][0] + a[c][1];
-#pragma unroll
-                for (int m = 4; m > 0; m >>= 1) {
-                    oo += __shfl_xor_sync(0xffffffffu, oo, m);
-                    if (DELTA) aa += __shfl_xor_sync(0xffffffffu, aa, m);
-                }
+                part[c][r] = sum2(o[c][0]) + sum2(o[c][1]);
                 if (DELTA) {
-                    const float uu = beta * (vr[c] - aa);
-                    oo = fmaf(uu, kq, oo);
+                    float aa = sum2(a[c][0]) + sum2(a[c][1]);
 #pragma unroll
-                    for (int e = 0; e < NE; ++e) {
-                        float* st = S[c] + 4 * e;
-                        st[0] = fmaf(k4[e].x, uu, st[0]); st[1] = fmaf(k4[e].y, uu, st[1]);
-                        st[2] = fmaf(k4[e].z, uu, st[2]); st[3] = fmaf(k4[e].w, uu, st[3]);
-                    }
+                    for (int m = 4; m > 0; m >>= 1) aa += __shfl_xor_sync(0xffffffffu, aa, m);
+                    const float uu = nums.x * (vr[c] - aa);
+                    if (p == r) oc[c] = uu * nums.y;
+                    const unsigned long long u2 = pack2(uu, uu);
+#pragma unroll
+                    for (int e = 0; e < 2 * NE; ++e) S[c][e] = fma2(k2[e], u2, S[c][e]);
                 }
-                if (p == r) oc[c] = oo;
+            }
+        };
+        if (rows == R) {                                      // a whole stage: no branch between its rows
+#pragma unroll
+            for (int r = 0; r < R; ++r) row(r);
+        } else {
+#pragma unroll
+            for (int r = 0; r < R; ++r) {
+                if (r < rows) row(r);
+                else
+#pragma unroll
+                    for (int c = 0; c < NC; ++c) part[c][r] = 0.f;
             }
         }
+#pragma unroll
+        for (int c = 0; c < NC; ++c) oc[c] += scatter_sum8(part[c], p);
         if (t0 + p < last) {
 #pragma unroll
             for (int c = 0; c < NC; ++c)
@@ -355,11 +465,11 @@ __global__ void __launch_bounds__(128) head_scan_kernel(HeadScan g, const T* __r
             const int d = 4 * p + 32 * e;
             float* dst = sp + (size_t)(col + c) * D + d;
             if (vec && col + c < g.vdim && d < D) {
-                *reinterpret_cast<float4*>(dst) = make_float4(S[c][4 * e], S[c][4 * e + 1], S[c][4 * e + 2], S[c][4 * e + 3]);
+                *reinterpret_cast<ulonglong2*>(dst) = make_ulonglong2(S[c][2 * e], S[c][2 * e + 1]);
             } else {
 #pragma unroll
                 for (int i = 0; i < 4; ++i)
-                    if (col + c < g.vdim && d + i < D) dst[i] = S[c][4 * e + i];
+                    if (col + c < g.vdim && d + i < D) dst[i] = __uint_as_float((unsigned)(S[c][2 * e + i / 2] >> (32 * (i & 1))));
             }
         }
     if (!DELTA || g.taps <= 1) return;

@@ -1775,7 +1775,7 @@ static void launch_head_scan(const HeadScan& g, const void* v, int batch, cudaSt
     if (ne <= 1) B200H_HS(1, 2);
     else if (ne <= 2) B200H_HS(2, 2);
     else if (ne <= 4) B200H_HS(4, 2);
-    else B200H_HS(8, 1);
+    else B200H_HS(8, 2);
 #undef B200H_HS
 }
 
@@ -1807,11 +1807,13 @@ static void launch_delta_prep(const b200h_delta_args* a, const DeltaPrep& d, cud
 {
     const bool vec = a->dim % 2 == 0 && (a->heads * a->vdim) % 2 == 0 && a->ld % 2 == 0 && reinterpret_cast<uintptr_t>(a->u) % (2 * sizeof(T)) == 0 &&
                      reinterpret_cast<uintptr_t>(a->conv) % 8 == 0 && reinterpret_cast<uintptr_t>(a->qkv) % 8 == 0;
-    const int v = vec ? 2 : 1, yb = a->kv_heads + (a->heads * a->vdim + 128 * v - 1) / (128 * v);
+    // a block's threads cover the query and key channels of `per` heads at once
+    const int v = vec ? 2 : 1, fit = 64 * v / a->dim, per = fit < 1 ? 1 : (fit > a->kv_heads ? a->kv_heads : fit), hb = (a->kv_heads + per - 1) / per;
+    const int yb = hb + (a->heads * a->vdim + 128 * v - 1) / (128 * v);
     const bool many = (int64_t)yb * a->n >= 8 * 1184 && a->taps <= 4;       // eight rows per block once that leaves eight blocks per SM
 #define B200H_DP(TAPS, ROWS, V)                                                                                                     \
-    delta_prep_kernel<T, TAPS, ROWS, V><<<dim3((a->n + ROWS - 1) / ROWS, yb), 128, (size_t)ROWS * 2 * a->dim * sizeof(float), st>>>( \
-        (const T*)a->u, (const T*)a->b, a->ld, d)
+    delta_prep_kernel<T, TAPS, ROWS, V><<<dim3((a->n + ROWS - 1) / ROWS, yb), 128, (size_t)ROWS * per * 2 * a->dim * sizeof(float), st>>>( \
+        (const T*)a->u, (const T*)a->b, a->ld, d, per, hb)
 #define B200H_DP_V(TAPS, ROWS) do { if (vec) B200H_DP(TAPS, ROWS, 2); else B200H_DP(TAPS, ROWS, 1); } while (0)
     if (a->taps <= 4) { if (many) B200H_DP_V(4, 8); else B200H_DP_V(4, 1); }
     else B200H_DP_V(B200H_MAX_TAPS, 1);
